@@ -122,13 +122,15 @@ class SequencePages:
     still see (the last W positions), so pages that fall wholly behind the window
     go back to the pool as the sequence grows; with `keep_first` = F the pages that
     hold any of the first F positions stay as well (a window that never loses the
-    sequence's first tokens).  Entry i of `table` is the page that holds positions
-    [i*PAGE_TOKENS, (i+1)*PAGE_TOKENS), or -1 once dropped.
+    sequence's first tokens).  `chunk` = C keeps only the pages of the chunk of C positions, counted from
+    position 0, that the next position lies in: the others go back when a chunk is through.  Entry i of
+    `table` is the page that holds positions [i*PAGE_TOKENS, (i+1)*PAGE_TOKENS), or -1 once dropped.
     """
 
-    def __init__(self, pool: PagePool, window: int = 0, keep_first: int = 0):
+    def __init__(self, pool: PagePool, window: int = 0, keep_first: int = 0, chunk: int = 0):
         self.pool = pool
         self.window = window
+        self.chunk = chunk
         self.keep_first = keep_first
         self.table: List[int] = []
         self.length = 0
@@ -145,8 +147,11 @@ class SequencePages:
         self.length += n_new
         if self.length > len(self.table) * PAGE_TOKENS:
             raise CacheMisuse("sequence advanced beyond its reserved pages")
-        if self.window > 0:
-            first_needed = max(0, self.length - self.window + 1) // PAGE_TOKENS
+        if self.window > 0 or self.chunk > 0:
+            first = max(0, self.length - self.window + 1) if self.window > 0 else 0
+            if self.chunk > 0:                   # the next position is `length`: its chunk's first position
+                first = max(first, self.length - self.length % self.chunk)
+            first_needed = min(first // PAGE_TOKENS, len(self.table))
             kept = pages_for(self.keep_first)
             drop = [p for p in self.table[kept:first_needed] if p >= 0]
             if drop:

@@ -38,6 +38,8 @@ class KVSpec:
     value_dim: Optional[int] = None
     # with a window: the first `keep_first` positions of a sequence stay visible (and held) whatever its length
     keep_first: int = 0
+    # C > 0: only keys of the next position's own chunk of C positions, counted from position 0, are kept
+    chunk: int = 0
 
     @property
     def v_heads(self) -> int:
@@ -55,7 +57,8 @@ class StateSpec:
     dtype: str = "float32"
 
 
-CacheSpec = Union[KVSpec, StateSpec]
+# a tuple: what several mixers of one stop keep, each for itself (a mixer made of mixers)
+CacheSpec = Union[KVSpec, StateSpec, Tuple[Union[KVSpec, StateSpec], ...]]
 
 
 @dataclass
@@ -67,6 +70,7 @@ class LayerCache:
     v: Optional[torch.Tensor] = None
     block_table: Optional[torch.Tensor] = None    # int32 [sequences in step, pages per sequence]
     state: Optional[torch.Tensor] = None          # [slots, *shape]; rows indexed by StepBatch.seq_slot
+    parts: Tuple["LayerCache", ...] = ()          # a tuple of specs: the view of each, in its order
 
 
 class _Group:
@@ -95,17 +99,22 @@ class SequenceCache:
         self.dtype, self.device = dtype, device
         self.slots = SlotTable(self.max_seqs)
         self.groups: List[_Group] = []
-        self.layer_group: Dict[int, Tuple[int, int]] = {}       # layer -> (group, index in group)
+        self.layer_group: Dict[int, Tuple[int, int]] = {}       # layer -> (group, index in group) of the first it keeps
+        self.layer_places: Dict[int, Tuple[Tuple[int, int], ...]] = {}    # the same of everything it keeps
+        self.layer_spec: Dict[int, CacheSpec] = {}
         by_spec: Dict[CacheSpec, int] = {}
-        for li, spec in enumerate(layer_specs):
-            if spec is None:
+        for li, specs in enumerate(layer_specs):
+            if specs is None:
                 continue
-            if spec not in by_spec:
-                by_spec[spec] = len(self.groups)
-                self.groups.append(_Group(spec))
-            g = self.groups[by_spec[spec]]
-            self.layer_group[li] = (by_spec[spec], len(g.layers))
-            g.layers.append(li)
+            places = []
+            for spec in specs if isinstance(specs, tuple) else (specs,):
+                if spec not in by_spec:
+                    by_spec[spec] = len(self.groups)
+                    self.groups.append(_Group(spec))
+                g = self.groups[by_spec[spec]]
+                places.append((by_spec[spec], len(g.layers)))
+                g.layers.append(li)
+            self.layer_group[li], self.layer_places[li], self.layer_spec[li] = places[0], tuple(places), specs
         for g in self.groups:
             if isinstance(g.spec, KVSpec):
                 g.pool = PagePool(self.n_pages)
@@ -142,8 +151,8 @@ class SequenceCache:
     # ------------------------------------------------------------------ sequences
     def acquire(self) -> int:
         slot = self.slots.acquire()
-        self._seq[slot] = [SequencePages(g.pool, g.spec.window, g.spec.keep_first) if isinstance(g.spec, KVSpec) else None
-                           for g in self.groups]
+        self._seq[slot] = [SequencePages(g.pool, g.spec.window, g.spec.keep_first, g.spec.chunk)
+                           if isinstance(g.spec, KVSpec) else None for g in self.groups]
         for g in self.groups:
             if g.state is not None:
                 g.state[:, slot].zero_()
@@ -235,7 +244,12 @@ class SequenceCache:
     def layer_view(self, layer: int, writes: bool, block_tables: Dict[int, torch.Tensor]) -> LayerCache:
         if layer not in self.layer_group:
             return LayerCache(spec=None, writes=False)
-        gi, idx = self.layer_group[layer]
+        views = tuple(self._view(place, writes, block_tables) for place in self.layer_places[layer])
+        spec = self.layer_spec[layer]
+        return LayerCache(spec=spec, writes=writes, parts=views) if isinstance(spec, tuple) else views[0]
+
+    def _view(self, place: Tuple[int, int], writes: bool, block_tables: Dict[int, torch.Tensor]) -> LayerCache:
+        gi, idx = place
         g = self.groups[gi]
         if isinstance(g.spec, KVSpec):
             return LayerCache(spec=g.spec, writes=writes, k=g.k[idx], v=None if g.v is None else g.v[idx],

@@ -1,5 +1,6 @@
 from .base import ConfigError, KeyReader, ModelConfig, read_config_json
 from .dabodra import DabodraConfig
+from .getizen import GetizenConfig
 from .llama import LlamaConfig, RopeScaling
 from .mokatar import MokatarConfig
 from .nibelorn import NibelornConfig
@@ -7,6 +8,6 @@ from .vitinex import VitinexConfig
 from .registry import (Architecture, architecture_name, find_architecture, register_architecture,
                        registered_architectures)
 
-__all__ = ["ConfigError", "KeyReader", "ModelConfig", "read_config_json", "LlamaConfig", "RopeScaling", "NibelornConfig", "DabodraConfig", "VitinexConfig", "MokatarConfig",
+__all__ = ["ConfigError", "KeyReader", "ModelConfig", "read_config_json", "LlamaConfig", "RopeScaling", "NibelornConfig", "DabodraConfig", "VitinexConfig", "MokatarConfig", "GetizenConfig",
            "Architecture", "architecture_name", "find_architecture", "register_architecture",
            "registered_architectures"]

@@ -10,10 +10,12 @@
 //   score_t    = (q[h][m] . K_t[kh]) * scale * temp(p),  temp(p) = 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)
 //   score_t   <- softcap * tanh(score_t / softcap)       (softcap > 0)
 //   a_m        = sum_t softmax_t(score) V_t[vh]           over the keys t in [lo, p], lo = 0 or p - window + 1,
-//                                                         and with a window also the keys t < keep_first
+//                                                         and with a window also the keys t < keep_first;
+//                                                         chunked (mask_chunk): only keys of p's own chunk of positions
+// head_scale: where given, one more factor per head on the score.
 // Values: rows of the value cache, or (v_in_k) the first v_dim values of the key rows of head (h / group) * maps.
 // sink: where given, exp(sink[h]) is one more term of every softmax's denominator (it has no key and no value).
-// combine 0 (maps = 1): out[h] = a_0.
+// combine 0 (maps = 1): out[h] = a_0, times sigmoid(gate[h * v_dim + d]) element by element where `gate` is given.
 // combine 1 (maps = 2): o = a_0 - lambda * a_1;  o <- o / sqrt(mean(o^2) + eps) * out_scale;
 //                       o <- o * sigmoid(gate[h]) where a gate column is given (gate: q's rows, column gate_col + h).
 //
@@ -46,8 +48,8 @@ attention_general_kernel(const GeneralAttention P) {
 
   float temp = 1.f;
   if (P.temp_coef != 0.f) temp = 1.f + P.temp_coef * logf((float)((pos + 1) / P.temp_every) + 1.f);
-  const float factor = P.scale * temp;
-  const int lo = (P.window > 0 && pos - P.window + 1 > 0) ? pos - P.window + 1 : 0;
+  const float factor = P.scale * temp * (P.head_scale ? P.head_scale[h] : 1.f);
+  const int lo = general_first_key(P, pos);
   // chunks are visited in key order: those that hold kept first keys, then those from the window's first key on
   const int first_win = (lo / 32) * 32;
   const int kept_end = min(P.window > 0 ? P.keep_first : 0, lo);
@@ -122,7 +124,10 @@ attention_general_kernel(const GeneralAttention P) {
 #pragma unroll
     for (int i = 0; i < VCH; i++) {
       const int d = lane + 32 * i;
-      if (d < Dv) op[d] = from_float<T>(acc[0][i] * inv);
+      if (d >= Dv) continue;
+      float r = acc[0][i] * inv;
+      if (P.gate) r /= 1.0f + expf(-P.gate[(size_t)t * P.ld_gate + (size_t)h * Dv + d]);
+      op[d] = from_float<T>(r);
     }
     return;
   }

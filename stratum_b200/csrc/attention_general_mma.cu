@@ -103,12 +103,12 @@ attention_general_mma_kernel(const GeneralAttention P) {
       row_pos[rg][e] = P.token_pos[row_tok[rg][e]];
       float temp = 1.f;
       if (P.temp_coef != 0.f) temp = 1.f + P.temp_coef * logf((float)((row_pos[rg][e] + 1) / P.temp_every) + 1.f);
-      row_factor[rg][e] = P.scale * temp;
+      row_factor[rg][e] = P.scale * temp * (P.head_scale ? P.head_scale[row_head[e]] : 1.f);
     }
   }
   const int first_pos = P.token_pos[tok0];
   const int last_pos = first_pos + ntok - 1;
-  const int lo_block = (P.window > 0 && first_pos - P.window + 1 > 0) ? first_pos - P.window + 1 : 0;
+  const int lo_block = general_first_key(P, first_pos), lo_last = general_first_key(P, last_pos);
   const int k_begin = split * P.chunk;
   const int k_end = min((split + 1) * P.chunk, last_pos + 1);
   // tiles wholly in front of the window of the block's first row hold nothing any row sees, unless they hold kept
@@ -210,12 +210,15 @@ attention_general_mma_kernel(const GeneralAttention P) {
         }
       }
     }
-    // a tile every row of the CTA sees whole (all of it at or before the first row's position, inside the item's
-    // range, no window) needs no mask: rows that do not exist carry zeros and are never written
-    const bool whole_tile = P.window == 0 && key0 + GM_TILE - 1 <= first_pos && key0 >= k_begin && key0 + GM_TILE <= k_end;
+    // a tile every row of the CTA sees whole (all of it at or before the first row's position, not in front of the
+    // last row's first key, inside the item's range) needs no mask: rows that do not exist carry zeros and are never
+    // written
+    const bool whole_tile = key0 >= lo_last && key0 + GM_TILE - 1 <= first_pos && key0 >= k_begin && key0 + GM_TILE <= k_end;
 #pragma unroll
     for (int rg = 0; rg < RG; rg++) {
       float bm[2] = {-INFINITY, -INFINITY};
+      int lo_of[2] = {0, 0};
+      if (!whole_tile) { lo_of[0] = general_first_key(P, row_pos[rg][0]); lo_of[1] = general_first_key(P, row_pos[rg][1]); }
 #pragma unroll
       for (int i = 0; i < 2; i++) {
 #pragma unroll
@@ -226,7 +229,7 @@ attention_general_mma_kernel(const GeneralAttention P) {
           if (!whole_tile) {
             const int key = kw + 8 * i + 2 * t + (j & 1);
             const int pos = row_pos[rg][e];
-            const int lo = (P.window > 0 && pos - P.window + 1 > 0) ? pos - P.window + 1 : 0;
+            const int lo = lo_of[e];
             const bool ok = any && row_ok[rg][e] && key <= pos && (key >= lo || key < keep) && key < k_end && key >= k_begin;
             v = ok ? v : -INFINITY;
           }
@@ -351,11 +354,21 @@ attention_general_mma_kernel(const GeneralAttention P) {
         for (int cc = 0; cc < CPW; cc++) {
           const int d = 32 * (warp + GM_WARPS * cc) + 8 * t;
           if (d >= Dv) continue;
+          float r[8];
+#pragma unroll
+          for (int i = 0; i < 8; i++) r[i] = o[rg][4 * cc + (i >> 1)][2 * e + (i & 1)] * inv;
+          if (P.gate) {
+            const float4* gp = reinterpret_cast<const float4*>(P.gate + (size_t)row_tok[rg][e] * P.ld_gate +
+                                                               (size_t)row_head[e] * Dv + d);
+            const float4 ga = gp[0], gb = gp[1];
+            r[0] /= 1.0f + expf(-ga.x); r[1] /= 1.0f + expf(-ga.y); r[2] /= 1.0f + expf(-ga.z); r[3] /= 1.0f + expf(-ga.w);
+            r[4] /= 1.0f + expf(-gb.x); r[5] /= 1.0f + expf(-gb.y); r[6] /= 1.0f + expf(-gb.z); r[7] /= 1.0f + expf(-gb.w);
+          }
           uint4 v;
-          v.x = pack_bf16(o[rg][4 * cc + 0][2 * e] * inv, o[rg][4 * cc + 0][2 * e + 1] * inv);
-          v.y = pack_bf16(o[rg][4 * cc + 1][2 * e] * inv, o[rg][4 * cc + 1][2 * e + 1] * inv);
-          v.z = pack_bf16(o[rg][4 * cc + 2][2 * e] * inv, o[rg][4 * cc + 2][2 * e + 1] * inv);
-          v.w = pack_bf16(o[rg][4 * cc + 3][2 * e] * inv, o[rg][4 * cc + 3][2 * e + 1] * inv);
+          v.x = pack_bf16(r[0], r[1]);
+          v.y = pack_bf16(r[2], r[3]);
+          v.z = pack_bf16(r[4], r[5]);
+          v.w = pack_bf16(r[6], r[7]);
           *reinterpret_cast<uint4*>(op + d) = v;
         }
       } else {
@@ -424,7 +437,9 @@ __global__ void __launch_bounds__(128) attention_general_finish_kernel(const Gen
       a[m] = acc;
     }
     if (MAPS == 1) {
-      op[d] = __float2bfloat16_rn(a[0]);
+      float r = a[0];
+      if (P.gate) r /= 1.0f + expf(-P.gate[(size_t)tok * P.ld_gate + (size_t)h * Dv + d]);
+      op[d] = __float2bfloat16_rn(r);
     } else {
       o[i] = a[0] - P.lambda * a[MAPS - 1];
       ss = fmaf(o[i], o[i], ss);
@@ -482,6 +497,7 @@ STRATUM_EXPORT int stratum_attention_general_mma(const GeneralAttention* params,
     return STRATUM_ERR_SHAPE;
   if ((((uintptr_t)P.q | (uintptr_t)P.out | (uintptr_t)P.k_cache | (uintptr_t)P.v_cache) & 15) != 0)
     return STRATUM_ERR_ALIGN;
+  if (P.gate && (P.ld_gate % 4 != 0 || ((uintptr_t)P.gate & 15) != 0)) return STRATUM_ERR_ALIGN;
   if (P.n_splits < 1 || P.n_splits > GM_MAX_SPLITS || P.v_dim > 512 || P.chunk < GM_TILE || P.chunk % GM_TILE != 0 || P.tokens_per_block < 1) return STRATUM_ERR_SHAPE;
   const bool direct = P.n_splits == 1 && P.combine == 0;
   if (!direct && (!P.part_o || !P.part_ml)) return STRATUM_ERR_SHAPE;

@@ -1,5 +1,5 @@
 // Gated linear attention: a recurrent mixer whose state is one matrix S [dim][vdim] per head, in float32, with a decay
-// per key channel.
+// per key channel; and retention, the same recurrence with one constant decay per head.
 //
 // Per token, from the float32 sums of the fused input projection (row = [q | k | v | g | a]: n_heads * dim twice,
 // n_heads * vdim twice, then `rank` values of the decay's inner projection):
@@ -10,7 +10,10 @@
 //   recur     per head, token after token:  S <- diag(alpha) S + k v^T;  o = S^T q * dim^(-1/2)
 //             (the decay acts on the rows of S, which belong to key channels; o sees the token's own write).
 //   finish    o / sqrt(mean_vdim(o^2) + eps) * gain * silu(g), rounded to the compute dtype for the output product.
-// All of it is float32 whatever the compute dtype.
+// With a constant decay per head (`head_decay`) there is no inner projection and neither cast nor decay; instead
+//   rotate    turns the first dimensions of every head of q and k, in place, by the step's table of cosines and sines,
+//             in pairs (i, i + pairs) or, interleaved, (2i, 2i + 1);
+// and the heads' norm may have no gain.  All of it is float32 whatever the compute dtype.
 //
 // The recurrence is sequential in the tokens of a sequence and independent across sequences, heads and columns of S:
 // a block owns (sequence, head, a tile of columns), a lane 16 rows of one column, so a column's read-out is split over
@@ -24,8 +27,8 @@
 struct Gla {
   const float* proj;        // [tokens][ld]
   void* inner;              // [tokens][ld_inner], the compute dtype: the decay's inner projection (cast)
-  const float* reserved_p;
-  const float* gain;        // [vdim]
+  const float* head_decay;  // [n_heads] or null: the decays are alpha's
+  const float* gain;        // [vdim] or null: none
   float* alpha;             // [tokens][n_heads * dim]: z when `decay` begins, alpha when it ends
   float* o_raw;             // [tokens][n_heads * vdim]
   void* out;                // [tokens][ldo] compute dtype
@@ -35,7 +38,7 @@ struct Gla {
   const int* seq_slot;      // [seqs]
   int ld, ldo, n_tokens, n_seqs;
   int n_heads, dim, vdim, rank;
-  int state_stride, write_state, ld_inner, reserved_i;
+  int state_stride, write_state, ld_inner, rot_pairs;
   float eps, inv_tau, q_scale, reserved;
 };
 
@@ -65,6 +68,25 @@ __global__ void __launch_bounds__(256) gla_decay_kernel(const Gla P) {
   }
 }
 
+// ---------------------------------------------------------------- rotate: a thread per (token, q or k, head, pair)
+__global__ void __launch_bounds__(256) gla_rotate_kernel(const Gla P, const float2* cs, int interleaved) {
+  pdl_trigger();
+  pdl_wait();                                        // the projection and the table are work of kernels before: ld_fresh
+  const int pairs = P.rot_pairs, per_token = 2 * P.n_heads * pairs;
+  const size_t n = (size_t)P.n_tokens * per_token;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = i / per_token;
+    const int rest = (int)(i - t * per_token), head = rest / pairs, pair = rest - head * pairs;    // q's heads, then k's
+    float* base = const_cast<float*>(P.proj) + t * P.ld + (size_t)head * P.dim;
+    float* pu = base + (interleaved ? 2 * pair : pair);
+    float* pv = base + (interleaved ? 2 * pair + 1 : pair + pairs);
+    const float2 f = __ldcg(cs + t * pairs + pair);
+    const float u = ld_fresh(pu), v = ld_fresh(pv);
+    *pu = u * f.x - v * f.y;
+    *pv = v * f.x + u * f.y;
+  }
+}
+
 // ---------------------------------------------------------------- the recurrence
 #define GLA_THREADS 128
 #define GLA_ROWS 16           // rows of a column of S that a lane holds
@@ -83,7 +105,8 @@ __device__ __forceinline__ void gla_wait_all() { asm volatile("cp.async.wait_all
 
 // The state of a head lies in memory column by column (S^T: [vdim][dim]), so the rows a lane holds are contiguous and
 // neighbouring lanes read neighbouring stretches.  A column is spread over L lanes of 16 rows each (dim <= 16 L).
-template <int L>
+// CONST_DECAY: the decay is the head's constant, and only k and q are staged.
+template <int L, bool CONST_DECAY>
 __global__ void __launch_bounds__(GLA_THREADS) gla_recur_kernel(const Gla P) {
   constexpr int ROWS = GLA_ROWS;
   constexpr int COLS = GLA_THREADS / L;
@@ -91,7 +114,8 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_recur_kernel(const Gla P) {
   constexpr int KQ = L * PITCH;                      // neighbouring lanes fall on different banks
   constexpr int FIT = 1280 / KQ;
   constexpr int CHUNK = FIT < 2 ? 2 : (FIT > GLA_MAX_CHUNK ? GLA_MAX_CHUNK : FIT);
-  __shared__ __align__(16) float kqa_s[2][CHUNK][3][KQ];      // k, q, alpha of the staged tokens
+  constexpr int STAGED = CONST_DECAY ? 2 : 3;
+  __shared__ __align__(16) float kqa_s[2][CHUNK][STAGED][KQ];      // k, q (, alpha) of the staged tokens
   __shared__ float v_s[2][CHUNK][COLS];
   const int seq = blockIdx.z, h = blockIdx.y, tile = blockIdx.x;
   const int r0 = P.seq_start[seq], r1 = P.seq_start[seq + 1];
@@ -122,24 +146,26 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_recur_kernel(const Gla P) {
     }
   }
   if (D != ROWS * L) {       // the dimensions beyond dim in the staging buffers stay zero: nothing below writes them
-    for (int i = threadIdx.x; i < 2 * CHUNK * 3 * KQ; i += GLA_THREADS) (&kqa_s[0][0][0][0])[i] = 0.f;
+    for (int i = threadIdx.x; i < 2 * CHUNK * STAGED * KQ; i += GLA_THREADS) (&kqa_s[0][0][0][0])[i] = 0.f;
     __syncthreads();
   }
 
+  const float hd = CONST_DECAY ? P.head_decay[h] : 0.f;
+  const float2 head_decay = make_float2(hd, hd);
   const bool vec_in = D % 4 == 0 && P.ld % 4 == 0 && ((((uintptr_t)P.proj) | ((uintptr_t)P.alpha)) & 15) == 0;
   auto stage = [&](int buf, int c0) {                // ask for the tokens c0 .. of this sequence
     const int n_here = min(CHUNK, r1 - c0);
     for (int tok = 0; tok < n_here; tok++) {
       const float* row = P.proj + (size_t)(c0 + tok) * P.ld + (size_t)h * D;
-      const float* al = P.alpha + (size_t)(c0 + tok) * HD + (size_t)h * D;
+      const float* al = CONST_DECAY ? nullptr : P.alpha + (size_t)(c0 + tok) * HD + (size_t)h * D;
       if (vec_in) {
-        for (int d = 4 * threadIdx.x; d < 3 * D; d += 4 * GLA_THREADS) {         // k, then q, then alpha
+        for (int d = 4 * threadIdx.x; d < STAGED * D; d += 4 * GLA_THREADS) {         // k, then q, then alpha
           const int which = d / D, dd = d - which * D;
           const float* src = which == 0 ? row + HD + dd : (which == 1 ? row + dd : al + dd);
           gla_copy16(&kqa_s[buf][tok][which][(dd / ROWS) * PITCH + dd % ROWS], src);
         }
       } else {
-        for (int d = threadIdx.x; d < 3 * D; d += GLA_THREADS) {
+        for (int d = threadIdx.x; d < STAGED * D; d += GLA_THREADS) {
           const int which = d / D, dd = d - which * D;
           const float* src = which == 0 ? row + HD + dd : (which == 1 ? row + dd : al + dd);
           gla_copy4(&kqa_s[buf][tok][which][(dd / ROWS) * PITCH + dd % ROWS], src);
@@ -165,15 +191,20 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_recur_kernel(const Gla P) {
     for (int tok = 0; tok < n_here; tok++, o_row += HV) {
       const float4* kk = reinterpret_cast<const float4*>(&kqa_s[buf][tok][0][part * PITCH]);
       const float4* qq = reinterpret_cast<const float4*>(&kqa_s[buf][tok][1][part * PITCH]);
-      const float4* aa = reinterpret_cast<const float4*>(&kqa_s[buf][tok][2][part * PITCH]);
+      const float4* aa = reinterpret_cast<const float4*>(&kqa_s[buf][tok][STAGED - 1][part * PITCH]);
       const float vj = v_s[buf][tok][col];
       const float2 vv = make_float2(vj, vj);
       float2 acc0 = make_float2(0.f, 0.f), acc1 = acc0;
 #pragma unroll
       for (int i = 0; i < ROWS / 4; i++) {
-        const float4 k4 = kk[i], q4 = qq[i], a4 = aa[i];
-        S[2 * i] = __ffma2_rn(make_float2(k4.x, k4.y), vv, __fmul2_rn(make_float2(a4.x, a4.y), S[2 * i]));
-        S[2 * i + 1] = __ffma2_rn(make_float2(k4.z, k4.w), vv, __fmul2_rn(make_float2(a4.z, a4.w), S[2 * i + 1]));
+        const float4 k4 = kk[i], q4 = qq[i];
+        float2 lo = head_decay, hi = head_decay;
+        if (!CONST_DECAY) {
+          const float4 a4 = aa[i];
+          lo = make_float2(a4.x, a4.y); hi = make_float2(a4.z, a4.w);
+        }
+        S[2 * i] = __ffma2_rn(make_float2(k4.x, k4.y), vv, __fmul2_rn(lo, S[2 * i]));
+        S[2 * i + 1] = __ffma2_rn(make_float2(k4.z, k4.w), vv, __fmul2_rn(hi, S[2 * i + 1]));
         acc0 = __ffma2_rn(S[2 * i], make_float2(q4.x, q4.y), acc0);
         acc1 = __ffma2_rn(S[2 * i + 1], make_float2(q4.z, q4.w), acc1);
       }
@@ -221,11 +252,11 @@ __global__ void __launch_bounds__(128) gla_finish_kernel(const Gla P) {
   ss = warp_sum(ss);
   const float mul = 1.0f / sqrtf(ss / (float)V + P.eps);
   for (int d = lane; d < V; d += 32)
-    out[d] = from_float<T>(ld_fresh(o + d) * mul * P.gain[d] * gla_silu(ld_fresh(g + d)));
+    out[d] = from_float<T>(ld_fresh(o + d) * mul * (P.gain ? P.gain[d] : 1.0f) * gla_silu(ld_fresh(g + d)));
 }
 
 static int gla_check(const Gla& P) {
-  if (P.n_heads < 1 || P.dim < 1 || P.vdim < 1 || P.rank < 1) return STRATUM_ERR_SHAPE;
+  if (P.n_heads < 1 || P.dim < 1 || P.vdim < 1 || P.rank < (P.head_decay ? 0 : 1)) return STRATUM_ERR_SHAPE;
   if (P.ld < 2 * P.n_heads * P.dim + 2 * P.n_heads * P.vdim + P.rank || P.ldo < P.n_heads * P.vdim)
     return STRATUM_ERR_SHAPE;
   if (P.state_stride < P.n_heads * P.dim * P.vdim) return STRATUM_ERR_SHAPE;
@@ -245,7 +276,7 @@ STRATUM_EXPORT int stratum_gla_cast(const Gla* params, int dtype, cudaStream_t s
   if (P.n_tokens <= 0) return 0;
   const int bad = gla_check(P);
   if (bad) return bad;
-  if (!P.inner || P.ld_inner < P.rank) return STRATUM_ERR_SHAPE;
+  if (!P.inner || P.ld_inner < P.rank || P.rank < 1) return STRATUM_ERR_SHAPE;
   const unsigned blocks = gla_blocks((size_t)P.n_tokens * P.rank);
   if (dtype == STRATUM_DT_F32) launch_pdl(gla_cast_kernel<float>, blocks, 256, 0, stream, P);
   else if (dtype == STRATUM_DT_BF16) launch_pdl(gla_cast_kernel<bf16>, blocks, 256, 0, stream, P);
@@ -253,11 +284,25 @@ STRATUM_EXPORT int stratum_gla_cast(const Gla* params, int dtype, cudaStream_t s
   return launch_status();
 }
 
+// Rotate q and k in place (one launch).  cs: [tokens][rot_pairs] (cos, sin).
+STRATUM_EXPORT int stratum_gla_rotate(const Gla* params, const void* cs, int interleaved, cudaStream_t stream) {
+  const Gla& P = *params;
+  if (P.n_tokens <= 0 || P.rot_pairs == 0) return 0;
+  const int bad = gla_check(P);
+  if (bad) return bad;
+  if (P.rot_pairs < 0 || 2 * P.rot_pairs > P.dim || !cs) return STRATUM_ERR_SHAPE;
+  if (((uintptr_t)cs & 7) != 0) return STRATUM_ERR_ALIGN;
+  launch_pdl(gla_rotate_kernel, gla_blocks((size_t)P.n_tokens * 2 * P.n_heads * P.rot_pairs), 256, 0, stream, P,
+             (const float2*)cs, interleaved);
+  return launch_status();
+}
+
 template <int L>
 static void gla_recur_launch(const Gla& P, cudaStream_t stream) {
   const int cols = GLA_THREADS / L;
   const dim3 grid((P.vdim + cols - 1) / cols, P.n_heads, P.n_seqs);
-  gla_recur_kernel<L><<<grid, GLA_THREADS, 0, stream>>>(P);
+  if (P.head_decay) gla_recur_kernel<L, true><<<grid, GLA_THREADS, 0, stream>>>(P);
+  else gla_recur_kernel<L, false><<<grid, GLA_THREADS, 0, stream>>>(P);
 }
 
 // The rest of a step, one launch each: which = 0 the decays from z (in place), 1 the recurrence, 2 finish.  dtype:

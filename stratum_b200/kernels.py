@@ -287,11 +287,13 @@ def gelu(x: torch.Tensor, kind: int = GELU_ERF) -> None:
     _check(f(_ptr(x), dtype_code(x.dtype), x.shape[0], x.shape[1], x.stride(0), kind, _stream()), "gelu")
 
 
-def swiglu(gu: torch.Tensor, out: torch.Tensor, act: int = 0) -> None:
-    """out[r][j] = silu(gu[r][2j]) * gu[r][2j+1]; with act (ACT_*), that activation takes silu's place."""
+def swiglu(gu: torch.Tensor, out: torch.Tensor, act: int = 0, limit: float = 0.0) -> None:
+    """out[r][j] = silu(gu[r][2j]) * gu[r][2j+1]; with act (ACT_*), that activation takes silu's place (limit:
+    ACT_CLAMPED_GATE's)."""
     _need(gu, "gu"); _need(out, "out", gu.dtype)
-    f = _fn("elementwise", "stratum_swiglu", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    _check(f(_ptr(gu), _ptr(out), dtype_code(gu.dtype), out.shape[0], out.shape[1], int(act), _stream()), "swiglu")
+    f = _fn("elementwise", "stratum_swiglu", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p])
+    _check(f(_ptr(gu), _ptr(out), dtype_code(gu.dtype), out.shape[0], out.shape[1], int(act), c_float(limit), _stream()),
+           "swiglu")
 
 
 def rope_store(qkv: torch.Tensor, token_pos: torch.Tensor, token_seq: torch.Tensor,
@@ -342,8 +344,9 @@ EPI_STORE, EPI_ADD_F32, EPI_STORE_F32, EPI_SWIGLU = 0, 1, 2, 3
 EPI_ADD_F32_EMIT, EPI_QKV_ROPE = 4, 5          # gemm_tc only: see GemmExtra
 
 
-# what a product with EPI_STORE may apply to what it stores; with EPI_SWIGLU: the gate's activation (0 = silu)
-ACT_NONE, ACT_GELU_ERF, ACT_GELU_TANH, ACT_RELU_SQ = 0, 1, 2, 3
+# what a product with EPI_STORE may apply to what it stores; with EPI_SWIGLU: the gate's activation (0 = silu).
+# ACT_CLAMPED_GATE (EPI_SWIGLU only, with a limit L): g sigmoid(1.702 g) (u + 1), g = min(gate, L), u = up in [-L, L]
+ACT_NONE, ACT_GELU_ERF, ACT_GELU_TANH, ACT_RELU_SQ, ACT_CLAMPED_GATE = 0, 1, 2, 3, 4
 
 
 def linear_simple(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
@@ -421,14 +424,15 @@ def _linear_shapes(x, w, bias, out, epilogue, what):
 
 
 def gemm_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
-                epilogue: int, act: int = ACT_NONE) -> None:
-    """bfloat16, at most 32 rows of x: the weight-streaming tensor-core kernel (see EPI_*; act as linear_simple's)."""
+                epilogue: int, act: int = ACT_NONE, limit: float = 0.0) -> None:
+    """bfloat16, at most 32 rows of x: the weight-streaming tensor-core kernel (see EPI_*; act as linear_simple's,
+    with EPI_SWIGLU the gate's; limit: ACT_CLAMPED_GATE's)."""
     M, N, Kd = _linear_shapes(x, w, bias, out, epilogue, "gemm_skinny")
     _need(x, "x", torch.bfloat16, contiguous=False)
     f = _fn("gemm_skinny", "stratum_gemm_skinny",
-            [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p])
     _check(f(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), epilogue, M, N, Kd, x.stride(0), out.stride(0), act,
-             _stream()), "gemm_skinny")
+             c_float(limit), _stream()), "gemm_skinny")
 
 
 _scratch_epoch = 0
@@ -491,7 +495,7 @@ class _EpiExtra(ctypes.Structure):
                 ("norm_parts", c_int), ("norm_ld", c_int), ("norm_size", c_float), ("norm_eps", c_float),
                 ("emit_ldx", c_int), ("emit_ld", c_int),
                 ("rope_pairs", c_int), ("bt_stride", c_int), ("n_q", c_int), ("n_kv", c_int), ("head_dim", c_int),
-                ("page_tokens", c_int), ("write_cache", c_int), ("act", c_int)]
+                ("page_tokens", c_int), ("write_cache", c_int), ("act", c_int), ("act_limit", c_float)]
 
 
 class GemmExtra:
@@ -504,15 +508,15 @@ class GemmExtra:
                   parts were written: `last_parts()` after the call);
     EPI_QKV_ROPE  the columns are query, key and value heads (pairs of rotated dimensions neighbours): queries
                   are rotated and stored to `out`, keys rotated and written, values written, into the paged cache;
-    activation    EPI_STORE applies ACT_* to what it stores.
+    activation    EPI_STORE applies ACT_* to what it stores, EPI_SWIGLU takes it for the gate's (limit: ACT_CLAMPED_GATE's).
     """
 
     def __init__(self):
         self.c = _EpiExtra()
         self.keep = []                      # tensors whose memory the struct points into
 
-    def activation(self, act: int) -> "GemmExtra":
-        self.c.act = int(act)
+    def activation(self, act: int, limit: float = 0.0) -> "GemmExtra":
+        self.c.act, self.c.act_limit = int(act), float(limit)
         return self
 
     def scaled_rows(self, norm_ss: torch.Tensor, parts: int, size: int, eps: float) -> "GemmExtra":
@@ -681,6 +685,7 @@ class _GeneralAttention(ctypes.Structure):
                 ("token_pos", c_void_p), ("token_seq", c_void_p), ("block_table", c_void_p),
                 ("qb_seq", c_void_p), ("qb_tok0", c_void_p), ("qb_ntok", c_void_p),
                 ("part_o", c_void_p), ("part_ml", c_void_p), ("seq_start", c_void_p), ("sink", c_void_p),
+                ("head_scale", c_void_p), ("gate", c_void_p),
                 ("ldq", c_int), ("ldo", c_int), ("bt_stride", c_int), ("n_tokens", c_int),
                 ("n_heads", c_int), ("group", c_int), ("maps", c_int),
                 ("qk_dim", c_int), ("v_dim", c_int), ("n_k_heads", c_int), ("n_v_heads", c_int), ("v_in_k", c_int),
@@ -688,6 +693,7 @@ class _GeneralAttention(ctypes.Structure):
                 ("temp_every", c_int), ("n_qblocks", c_int), ("tokens_per_block", c_int), ("n_splits", c_int),
                 ("chunk", c_int), ("reserved", c_int),
                 ("dense", c_int), ("ldk", c_int), ("ldv", c_int), ("keep_first", c_int),
+                ("mask_chunk", c_int), ("ld_gate", c_int),
                 ("scale", c_float), ("softcap", c_float), ("temp_coef", c_float), ("lam", c_float),
                 ("out_scale", c_float), ("eps", c_float)]
 
@@ -696,24 +702,32 @@ class AttentionShape:
     """The constants of a general attention (see csrc/attention_general.cu): heads, query heads per key/value
     head (`group`), score maps per head, key and value sizes, whether the values are the first v_dim values of
     the key rows, scale, softcap (0: none), window (0: every key; keep_first: with a window, the positions below it stay
-    visible), the query factor
+    visible), chunk (0: none; else a position sees only keys of its own chunk of that many positions, counted from
+    position 0), head_scale (float32 [n_heads] or None: a factor on the scores of each head), the query factor
     1 + temp_coef ln(floor((p + 1) / temp_every) + 1), and for two maps the combination
     (a_0 - lam a_1) / rms * out_scale with its eps and the column of the output gate (-1: none)."""
 
     def __init__(self, n_heads: int, group: int, maps: int, qk_dim: int, v_dim: int, v_in_k: bool, scale: float,
                  softcap: float = 0.0, window: int = 0, temp_coef: float = 0.0, temp_every: int = 1,
                  lam: float = 0.0, out_scale: float = 1.0, eps: float = 0.0, gate_col: int = -1,
-                 sink: Optional[torch.Tensor] = None, keep_first: int = 0):
+                 sink: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0,
+                 head_scale: Optional[torch.Tensor] = None):
         self.keep_first = int(keep_first) if window > 0 else 0
         self.n_heads, self.group, self.maps, self.qk_dim, self.v_dim = n_heads, group, maps, qk_dim, v_dim
         self.v_in_k, self.scale, self.softcap, self.window = bool(v_in_k), scale, softcap, window
         self.temp_coef, self.temp_every, self.lam, self.out_scale = temp_coef, temp_every, lam, out_scale
         self.eps, self.gate_col = eps, gate_col
-        if sink is not None:
-            _need(sink, "sink", torch.float32)
-            if sink.numel() != n_heads:
-                raise KernelError("attention: one sink per head")
-        self.sink = sink
+        for name, t in (("sink", sink), ("head_scale", head_scale)):
+            if t is not None:
+                _need(t, name, torch.float32)
+                if t.numel() != n_heads:
+                    raise KernelError(f"attention: one {name} per head")
+        self.sink, self.head_scale, self.chunk = sink, head_scale, int(chunk)
+
+    @property
+    def span(self) -> int:
+        """The most keys a row sees beside kept first ones (0: all)."""
+        return min(v for v in (self.window, self.chunk) if v > 0) if self.window > 0 or self.chunk > 0 else 0
 
     def fill(self, p: "_GeneralAttention") -> None:
         p.n_heads, p.group, p.maps, p.qk_dim, p.v_dim = self.n_heads, self.group, self.maps, self.qk_dim, self.v_dim
@@ -723,6 +737,16 @@ class AttentionShape:
         p.temp_every, p.scale, p.softcap, p.temp_coef = self.temp_every, self.scale, self.softcap, self.temp_coef
         p.lam, p.out_scale, p.eps, p.keep_first = self.lam, self.out_scale, self.eps, self.keep_first
         p.sink = None if self.sink is None else self.sink.data_ptr()
+        p.head_scale = None if self.head_scale is None else self.head_scale.data_ptr()
+        p.mask_chunk = self.chunk
+
+
+def _output_gate(p: "_GeneralAttention", gate: Optional[torch.Tensor]) -> None:
+    if gate is not None:
+        _need(gate, "gate", torch.float32, contiguous=False)
+        if gate.shape[0] != p.n_tokens or gate.shape[1] < p.n_heads * p.v_dim or gate.stride(1) != 1:
+            raise KernelError("attention: the output gate has a column per head and value dimension")
+        p.gate, p.ld_gate = gate.data_ptr(), gate.stride(0)
 
 
 def _general_params(shape: AttentionShape, q, k_cache, v_cache, token_pos, token_seq, block_table, out,
@@ -757,19 +781,23 @@ def _general_params(shape: AttentionShape, q, k_cache, v_cache, token_pos, token
 
 def attention_general(shape: AttentionShape, q: torch.Tensor, k_cache: torch.Tensor, v_cache: Optional[torch.Tensor],
                       token_pos: torch.Tensor, token_seq: torch.Tensor, block_table: torch.Tensor, out: torch.Tensor,
-                      page_tokens: int) -> None:
+                      page_tokens: int, gate: Optional[torch.Tensor] = None) -> None:
     """Causal attention of every token of the step over its sequence's cached keys for the shapes AttentionShape
-    describes, on the CUDA cores in float32 (q, the cache and out in one dtype)."""
+    describes, on the CUDA cores in float32 (q, the cache and out in one dtype).  gate (float32 [tokens, heads *
+    v_dim], one map only): the output times sigmoid(gate), element by element."""
     p = _general_params(shape, q, k_cache, v_cache, token_pos, token_seq, block_table, out, page_tokens)
+    _output_gate(p, gate)
     f = _fn("attention_general", "stratum_attention_general", [c_void_p, c_int, c_void_p])
     _check(f(ctypes.addressof(p), dtype_code(q.dtype), _stream()), "attention_general")
 
 
-def attention_general_mma_ok(shape: AttentionShape, q: torch.Tensor, out: torch.Tensor, page_tokens: int) -> bool:
+def attention_general_mma_ok(shape: AttentionShape, q: torch.Tensor, out: torch.Tensor, page_tokens: int,
+                             gate: Optional[torch.Tensor] = None) -> bool:
     """Whether the tensor-core form of the general attention takes this call (else: attention_general)."""
     return (q.dtype == torch.bfloat16 and shape.qk_dim % 8 == 0 and shape.v_dim % 8 == 0 and shape.v_dim <= 512
             and q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
-            and out.data_ptr() % 16 == 0 and page_tokens == 64)
+            and out.data_ptr() % 16 == 0 and page_tokens == 64
+            and (gate is None or (gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0)))
 
 
 def attention_general_mma_row_groups(v_dim: int) -> int:
@@ -782,7 +810,7 @@ def attention_general_mma(shape: AttentionShape, q: torch.Tensor, k_cache: torch
                           block_table: torch.Tensor, out: torch.Tensor, page_tokens: int, qblocks,
                           tokens_per_block: int, n_splits: int, chunk: int, part_o: Optional[torch.Tensor],
                           part_ml: Optional[torch.Tensor], row_groups: int = 1,
-                          seq_start: Optional[torch.Tensor] = None) -> None:
+                          seq_start: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
     """The general attention in bfloat16 on tensor cores.  qblocks: None (one token per sequence, block i is row i)
     or (seq, first row, tokens) int32 tensors with tokens <= row_groups * tokens_per_block, where
     tokens_per_block = 16 // min(group, 16) tokens make one group of 16 rows and row_groups is 1 or
@@ -791,8 +819,10 @@ def attention_general_mma(shape: AttentionShape, q: torch.Tensor, k_cache: torch
     more than one map the items' results go through scratch: part_o float32 [tokens*heads*maps*n_splits*v_dim],
     part_ml float32 [tokens*heads*maps*n_splits*2].  seq_start (int32, the first row of every sequence of the step):
     k_cache and v_cache are then plain matrices [rows, heads * size] that hold sequence s's keys and values by
-    position from row seq_start[s] on, with 64 readable rows beyond the last sequence's; no block table."""
+    position from row seq_start[s] on, with 64 readable rows beyond the last sequence's; no block table.  gate: as
+    attention_general's."""
     p = _general_params(shape, q, k_cache, v_cache, token_pos, token_seq, block_table, out, page_tokens, seq_start)
+    _output_gate(p, gate)
     if qblocks is None:
         p.n_qblocks = q.shape[0]
     else:
@@ -1045,12 +1075,12 @@ def ssm_scan(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, a_l
 # ------------------------------------------------------------------ gated linear attention
 class _Gla(ctypes.Structure):
     """Mirror of struct Gla in csrc/gla.cu."""
-    _fields_ = [("proj", c_void_p), ("inner", c_void_p), ("reserved_p", c_void_p), ("gain", c_void_p),
+    _fields_ = [("proj", c_void_p), ("inner", c_void_p), ("head_decay", c_void_p), ("gain", c_void_p),
                 ("alpha", c_void_p), ("o_raw", c_void_p), ("out", c_void_p), ("state", c_void_p),
                 ("token_seq", c_void_p), ("seq_start", c_void_p), ("seq_slot", c_void_p),
                 ("ld", c_int), ("ldo", c_int), ("n_tokens", c_int), ("n_seqs", c_int),
                 ("n_heads", c_int), ("dim", c_int), ("vdim", c_int), ("rank", c_int),
-                ("state_stride", c_int), ("write_state", c_int), ("ld_inner", c_int), ("reserved_i", c_int),
+                ("state_stride", c_int), ("write_state", c_int), ("ld_inner", c_int), ("rot_pairs", c_int),
                 ("eps", c_float), ("inv_tau", c_float), ("q_scale", c_float), ("reserved", c_float)]
 
 
@@ -1060,10 +1090,13 @@ class GlaStep:
     inner projection in a matrix of the compute dtype [tokens, >= rank]; the caller's matrix product turns it into z
     float32 [tokens, heads * dim]; `decay(z)` makes the decays of z in place; `recur(...)` runs the recurrence over
     every sequence's state (float32 [slots, >= heads * vdim * dim], S^T) and leaves the read-outs in o_raw float32
-    [tokens, heads * vdim]; `finish(...)` norms and gates them into out (compute dtype [tokens, >= heads * vdim])."""
+    [tokens, heads * vdim]; `finish(...)` norms and gates them into out (compute dtype [tokens, >= heads * vdim]).
+
+    With head_decay (float32 [heads]: a constant decay per head; rank 0) there is neither `cast` nor `decay`;
+    `rotate(table, interleaved)` turns q and k in place by the step's (cos, sin) table float32 [tokens, pairs, 2]."""
 
     def __init__(self, proj: torch.Tensor, n_heads: int, dim: int, vdim: int, rank: int, tau: float, q_scale: float,
-                 eps: float):
+                 eps: float, head_decay: Optional[torch.Tensor] = None):
         _need(proj, "proj", torch.float32, contiguous=False)
         p = self.p = _Gla()
         p.proj, p.ld, p.n_tokens = proj.data_ptr(), proj.stride(0), proj.shape[0]
@@ -1073,6 +1106,20 @@ class GlaStep:
         p.eps, p.inv_tau, p.q_scale = float(eps), 1.0 / float(tau), float(q_scale)
         p.n_seqs = 1
         self.T, self.keep = proj.shape[0], [proj]
+        if head_decay is not None:
+            _need(head_decay, "head_decay", torch.float32)
+            if head_decay.numel() != n_heads:
+                raise KernelError("gla: one decay per head")
+            p.head_decay = head_decay.data_ptr()
+            self.keep.append(head_decay)
+
+    def rotate(self, table: torch.Tensor, interleaved: bool) -> None:
+        _need(table, "table", torch.float32)
+        if table.dim() != 3 or table.shape[0] != self.T or table.shape[2] != 2:
+            raise KernelError("gla: the rotation's table is [tokens, pairs, 2]")
+        self.p.rot_pairs = table.shape[1]
+        f = _fn("gla", "stratum_gla_rotate", [c_void_p, c_void_p, c_int, c_void_p])
+        _check(f(ctypes.addressof(self.p), _ptr(table), int(bool(interleaved)), _stream()), "gla_rotate")
 
     def cast(self, inner: torch.Tensor) -> None:
         _need(inner, "inner", contiguous=False)
@@ -1100,20 +1147,157 @@ class GlaStep:
         _need(token_seq, "token_seq", torch.int32); _need(seq_start, "seq_start", torch.int32)
         _need(seq_slot, "seq_slot", torch.int32)
         p = self.p
-        if o_raw.shape != (self.T, p.n_heads * p.vdim) or state.dim() != 2 or not p.alpha:
+        if o_raw.shape != (self.T, p.n_heads * p.vdim) or state.dim() != 2 or not (p.alpha or p.head_decay):
             raise KernelError("gla: shapes disagree, or the decays were not made")
         p.o_raw, p.state, p.state_stride = o_raw.data_ptr(), state.data_ptr(), state.stride(0)
         p.token_seq, p.seq_start, p.seq_slot = token_seq.data_ptr(), seq_start.data_ptr(), seq_slot.data_ptr()
         p.n_seqs, p.write_state = seq_slot.numel(), int(bool(write_state))
         self._run(1, torch.float32, "gla_recur")
 
-    def finish(self, gain: torch.Tensor, out: torch.Tensor) -> None:
-        _need(gain, "gain", torch.float32); _need(out, "out", contiguous=False)
+    def finish(self, gain: Optional[torch.Tensor], out: torch.Tensor) -> None:
+        """gain: float32 [vdim], or None: the norm has no weight."""
+        _need(out, "out", contiguous=False)
+        if gain is not None:
+            _need(gain, "gain", torch.float32)
         p = self.p
-        if gain.numel() != p.vdim or out.shape[0] != self.T or out.shape[1] < p.n_heads * p.vdim or not p.o_raw:
+        if (gain is not None and gain.numel() != p.vdim) or out.shape[0] != self.T or out.shape[1] < p.n_heads * p.vdim or not p.o_raw:
             raise KernelError("gla: shapes disagree, or the recurrence has not run")
-        p.gain, p.out, p.ldo = gain.data_ptr(), out.data_ptr(), out.stride(0)
+        p.gain = None if gain is None else gain.data_ptr()
+        p.out, p.ldo = out.data_ptr(), out.stride(0)
         self._run(2, out.dtype, "gla_finish")
+
+
+# ------------------------------------------------------------------ the norm of a sum
+SUM_NORM_TERMS = 2
+
+
+class _SumNorm(ctypes.Structure):
+    """Mirror of struct SumNorm in csrc/sum_norm.cu."""
+    _fields_ = [("x", c_void_p), ("rows", c_void_p), ("y", c_void_p * SUM_NORM_TERMS),
+                ("y_gain", c_void_p * SUM_NORM_TERMS), ("gain", c_void_p), ("out", c_void_p), ("copy", c_void_p),
+                ("n_rows", c_int), ("hidden", c_int), ("groups", c_int), ("n_terms", c_int),
+                ("scale", c_float), ("eps", c_float), ("y_eps", c_float * SUM_NORM_TERMS), ("reserved", c_int)]
+
+
+def sum_norm(x: torch.Tensor, scale: float, terms, gain: Optional[torch.Tensor], groups: int, eps: float,
+             out: torch.Tensor, copy: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None) -> None:
+    """out = norm(scale * x + the sum of the terms), float32 [rows, H] inside (see csrc/sum_norm.cu).  terms: up to
+    SUM_NORM_TERMS objects with y (float32 [rows, H]), gain (float32 [H], or None: y is added as it is) and eps.  groups:
+    equal parts of a row that are normalised each by itself (0: no norm, gain and eps unused).  out: float32 (it may be
+    x) or bfloat16; copy (bfloat16): the same rows rounded; rows (int32): which rows of x to take (no terms then)."""
+    _need(x, "x", torch.float32); _need(out, "out")
+    H = x.shape[-1]
+    n = x.shape[0] if rows is None else rows.numel()
+    if out.shape != (n, H) or len(terms) > SUM_NORM_TERMS or (rows is not None and len(terms)):
+        raise KernelError("sum_norm: shapes disagree")
+    p = _SumNorm()
+    p.x, p.out, p.n_rows, p.hidden, p.groups, p.n_terms = x.data_ptr(), out.data_ptr(), n, H, int(groups), len(terms)
+    p.scale, p.eps = float(scale), float(eps)
+    if groups:
+        _need(gain, "gain", torch.float32)
+        if gain.numel() != H or H % groups:
+            raise KernelError("sum_norm: gain or groups and the row disagree")
+        p.gain = gain.data_ptr()
+    for j, t in enumerate(terms):
+        _need(t.y, "y", torch.float32)
+        if t.y.shape != (n, H):
+            raise KernelError("sum_norm: a term's shape and the stream's disagree")
+        p.y[j], p.y_eps[j] = t.y.data_ptr(), float(t.eps)
+        if t.gain is not None:
+            _need(t.gain, "y_gain", torch.float32)
+            if t.gain.numel() != H:
+                raise KernelError("sum_norm: a term's gain and the row disagree")
+            p.y_gain[j] = t.gain.data_ptr()
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+        p.rows = rows.data_ptr()
+    if copy is not None:
+        _need(copy, "copy", torch.bfloat16)
+        if copy.shape != (n, H):
+            raise KernelError("sum_norm: copy and the stream disagree")
+        p.copy = copy.data_ptr()
+    f = _fn("sum_norm", "stratum_sum_norm", [c_void_p, c_int, c_void_p])
+    _check(f(ctypes.addressof(p), dtype_code(out.dtype), _stream()), "sum_norm")
+
+
+# ------------------------------------------------------------------ the gated linear recurrence
+class _Lru(ctypes.Structure):
+    """Mirror of struct Lru in csrc/lru.cu."""
+    _fields_ = [("y", c_void_p), ("x", c_void_p), ("conv_w", c_void_p), ("conv_b", c_void_p), ("gate_w", c_void_p),
+                ("gate_b", c_void_p), ("rate", c_void_p), ("u", c_void_p), ("pre", c_void_p), ("out", c_void_p),
+                ("state", c_void_p), ("token_pos", c_void_p), ("token_seq", c_void_p), ("seq_start", c_void_p),
+                ("seq_slot", c_void_p),
+                ("ld", c_int), ("ldo", c_int), ("n_tokens", c_int), ("n_seqs", c_int), ("width", c_int),
+                ("blocks", c_int), ("taps", c_int), ("state_stride", c_int), ("write_state", c_int), ("max_new", c_int)]
+
+
+class LinearRecurrence:
+    """The weights of a gated linear recurrence and its launches (see csrc/lru.cu): conv_w float32 [taps, width] (the last
+    row is the current token's), conv_b [width], gates float32 or bfloat16 [blocks, 2 size, size] (the rows of r, then
+    those of i, of every block), gate_b [blocks, 2 size], rate [width] (log a = rate * r).  bfloat16 matrices whose size
+    is a multiple of 8 go to the tensor cores, against float32 rows in two bfloat16 parts; others to the CUDA cores."""
+
+    def __init__(self, conv_w: torch.Tensor, conv_b: torch.Tensor, gates: torch.Tensor, gate_b: torch.Tensor,
+                 rate: torch.Tensor):
+        for name, t in (("conv_w", conv_w), ("conv_b", conv_b), ("gate_b", gate_b), ("rate", rate)):
+            _need(t, name, torch.float32)
+        _need(gates, "gates")
+        self.taps, self.width = conv_w.shape
+        self.blocks, two, self.size = gates.shape
+        if two != 2 * self.size or self.blocks * self.size != self.width or gate_b.numel() != 2 * self.width \
+                or conv_b.numel() != self.width or rate.numel() != self.width:
+            raise KernelError("linear recurrence: the weights disagree")
+        self.tensor_cores = gates.dtype == torch.bfloat16 and self.size % 8 == 0
+        self.gates = gates if self.tensor_cores else gates.float()
+        self.conv_w, self.conv_b, self.gate_b, self.rate = conv_w, conv_b, gate_b, rate
+
+    def _params(self, proj, out, state, step, write_state: bool) -> "_Lru":
+        _need(proj, "proj", torch.float32, contiguous=False); _need(out, "out", contiguous=False)
+        _need(state, "state", torch.float32)
+        for name, t in (("token_pos", step.token_pos), ("token_seq", step.token_seq), ("seq_start", step.seq_start),
+                        ("seq_slot", step.seq_slot)):
+            _need(t, name, torch.int32)
+        W, T = self.width, proj.shape[0]
+        if proj.shape[1] < 2 * W or out.shape[0] != T or out.shape[1] < W or state.shape[1] < (1 + self.taps) * W:
+            raise KernelError("linear recurrence: buffers and sizes disagree")
+        p = _Lru()
+        p.y, p.x = proj.data_ptr(), proj.data_ptr() + 4 * W
+        p.conv_w, p.conv_b, p.gate_b, p.rate = (self.conv_w.data_ptr(), self.conv_b.data_ptr(), self.gate_b.data_ptr(),
+                                                self.rate.data_ptr())
+        p.out, p.state, p.state_stride = out.data_ptr(), state.data_ptr(), state.stride(0)
+        p.token_pos, p.token_seq = step.token_pos.data_ptr(), step.token_seq.data_ptr()
+        p.seq_start, p.seq_slot = step.seq_start.data_ptr(), step.seq_slot.data_ptr()
+        p.ld, p.ldo, p.n_tokens, p.n_seqs = proj.stride(0), out.stride(0), T, step.seq_slot.numel()
+        p.width, p.blocks, p.taps = W, self.blocks, self.taps
+        p.write_state, p.max_new = int(bool(write_state)), int(step.max_new)
+        return p
+
+    def run(self, runtime, proj: torch.Tensor, out: torch.Tensor, state: torch.Tensor, step, write_state: bool) -> None:
+        """proj float32 [tokens, >= 2 width]: the y branch before its activation, then the x branch before the
+        convolution; out (compute dtype [tokens, >= width]) = S * gelu_tanh(y); state float32 [slots, >= (1 + taps)
+        width]."""
+        p = self._params(proj, out, state, step, write_state)
+        p.gate_w = self.gates.data_ptr()
+        tc = self.tensor_cores
+        if tc and (proj.stride(0) % 4 or proj.data_ptr() % 16):
+            raise KernelError("linear recurrence: rows of the projection must be 16-byte aligned")
+        if tc and step.all_single and out.dtype == torch.bfloat16:
+            f = _fn("lru", "stratum_lru_step", [c_void_p, c_void_p])
+            _check(f(ctypes.addressof(p), _stream()), "lru_step")
+            return
+        T, W = proj.shape[0], self.width
+        u = runtime.empty(T, W, dtype=torch.float32)
+        pre = runtime.empty(T, 2 * W, dtype=torch.float32)
+        p.u, p.pre = u.data_ptr(), pre.data_ptr()
+        f = _fn("lru", "stratum_lru_conv", [c_void_p, c_void_p])
+        _check(f(ctypes.addressof(p), _stream()), "lru_conv")
+        if tc:
+            f = _fn("lru", "stratum_lru_gates", [c_void_p, c_void_p])
+            _check(f(ctypes.addressof(p), _stream()), "lru_gates")
+        else:
+            linear_heads(u, self.gates, pre, self.size, 2 * self.size)
+        f = _fn("lru", "stratum_lru_scan", [c_void_p, c_int, c_void_p])
+        _check(f(ctypes.addressof(p), dtype_code(out.dtype), _stream()), "lru_scan")
 
 
 # ------------------------------------------------------------------ routed experts

@@ -115,16 +115,17 @@ def run_general_dense(att, shape, q: torch.Tensor, keys: torch.Tensor, values: t
                             seq_start=step.seq_start)
 
 
-def run_general(att, shape, q: torch.Tensor, cache, step, out: torch.Tensor) -> None:
+def run_general(att, shape, q: torch.Tensor, cache, step, out: torch.Tensor, gate=None) -> None:
     """Attention of the shapes kernels.AttentionShape describes (key and value sizes of their own, values inside the
     key rows, several maps per head): q [tokens, *] holds head j's map m at column (j * maps + m) * qk_dim.
     bfloat16 with sizes in multiples of 8: the tensor-core kernel (decode steps: the keys cut into ranges that
     fill the GPU; prompts: query blocks of 16 rows); everything else: the CUDA-core kernel, float32 throughout.
+    gate (float32 [tokens, heads * v_dim] or None): pre-activations of an output gate per element.
     STRATUM_GENERAL_ATTENTION_MMA=0: always the CUDA-core kernel (measurements)."""
-    if (not K.attention_general_mma_ok(shape, q, out, PAGE_TOKENS)
+    if (not K.attention_general_mma_ok(shape, q, out, PAGE_TOKENS, gate)
             or os.environ.get("STRATUM_GENERAL_ATTENTION_MMA", "1") == "0"):
         K.attention_general(shape, q, cache.k, cache.v, step.token_pos, step.token_seq, cache.block_table, out,
-                            PAGE_TOKENS)
+                            PAGE_TOKENS, gate)
         return
     rows_per_token = min(shape.group, 16)
     per_block = 16 // rows_per_token
@@ -132,7 +133,7 @@ def run_general(att, shape, q: torch.Tensor, cache, step, out: torch.Tensor) -> 
     row_groups = 1
     if step.all_single:
         qblocks = None
-        n_splits, chunk = plan_general_splits(step.n_tokens * streams, step.max_len, shape.window)
+        n_splits, chunk = plan_general_splits(step.n_tokens * streams, step.max_len, shape.span)
     else:
         # prompts: a CTA takes several groups of 16 rows through every tile of keys, which then comes from L2 once
         row_groups = K.attention_general_mma_row_groups(shape.v_dim)
@@ -144,4 +145,4 @@ def run_general(att, shape, q: torch.Tensor, cache, step, out: torch.Tensor) -> 
         part_o = att.runtime.scratch("general_attention_part_o", n * shape.v_dim, torch.float32)
         part_ml = att.runtime.scratch("general_attention_part_ml", n * 2, torch.float32)
     K.attention_general_mma(shape, q, cache.k, cache.v, step.token_pos, step.token_seq, cache.block_table, out,
-                            PAGE_TOKENS, qblocks, per_block, n_splits, chunk, part_o, part_ml, row_groups)
+                            PAGE_TOKENS, qblocks, per_block, n_splits, chunk, part_o, part_ml, row_groups, gate=gate)

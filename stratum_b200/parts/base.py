@@ -13,7 +13,7 @@ Data conventions during a step:
 """
 from __future__ import annotations
 
-from typing import Any, Dict, Mapping, Optional
+from typing import Any, Dict, List, Mapping, Optional, Sequence, Tuple
 
 import torch
 
@@ -116,10 +116,24 @@ class Norm(Part):
         residual rows rounded.  Optional."""
         raise NotImplementedError(f"norm {self.kind!r} has no form that adds into the residual stream")
 
+    def norm_sum(self, x: torch.Tensor, terms: "Sequence[Term]", copy: Optional[torch.Tensor] = None) -> None:
+        """The form of a norm that takes the sum of the stream and a sublayer's output: x = norm(c x + the sum of the
+        terms), in place, float32 [T, hidden], c a constant of the norm; copy, where given (bfloat16), receives the new
+        rows rounded.  Optional."""
+        raise NotImplementedError(f"norm {self.kind!r} has no form over a sum")
+
     def forward_heads(self, x: torch.Tensor, first_col: int, n_heads: int, head_dim: int) -> None:
         """Normalise in place, in every row of x (compute dtype), each of the n_heads stretches of head_dim
         values that start at column first_col: the form a mixer uses on its queries and keys.  Optional."""
         raise NotImplementedError(f"norm {self.kind!r} has no per-head form")
+
+
+class Term:
+    """One summand of a sublayer's output that whoever adds it up still has to normalise: y (float32 [T, hidden]) over
+    its rows' root mean square (eps inside the root) times `gain` (float32 [hidden]); gain None: y as it is."""
+
+    def __init__(self, y: torch.Tensor, gain: Optional[torch.Tensor] = None, eps: float = 0.0):
+        self.y, self.gain, self.eps = y, gain, eps
 
 
 class PositionEncoding(Part):
@@ -150,12 +164,26 @@ class RotaryTable:
 
 
 class Mixer(Part):
+    # `terms(xn, step, cache)` gives the output as a list of Terms in place of adding it up: an arrangement whose next
+    # kernel reads the output anyway then adds the terms there
+    gives_terms = False
+    # `input_weights(weights)` gives the matrix (and bias or None) of the one product that reads the mixer's input, and
+    # forward takes `proj`, its float32 result [T, rows of the matrix]: a mixer made of mixers that read the same input
+    # runs their products as one (and binds them with own_projection=False)
+    splits_projection = False
+
     def cache_spec(self) -> Optional[CacheSpec]:
         """What this mixer keeps per sequence between steps (keys and values, fixed-size state, nothing)."""
         return None
 
     def forward(self, xn: torch.Tensor, residual: torch.Tensor, step, cache: LayerCache) -> None:
         """residual += mix(xn).  xn: compute dtype [T, hidden]; residual: float32 [T, hidden]."""
+        raise NotImplementedError
+
+    def terms(self, xn: torch.Tensor, step, cache: LayerCache) -> List[Term]:
+        raise NotImplementedError
+
+    def input_weights(self, weights: Mapping[str, torch.Tensor]) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
         raise NotImplementedError
 
 

@@ -5,7 +5,7 @@ import torch
 
 from .. import kernels as K
 from ..cache.store import LayerCache
-from .base import Arrangement
+from .base import Arrangement, Term
 from .registry import register_part
 
 
@@ -126,6 +126,55 @@ class OutputNormResidual(Arrangement):
         self._run(ff, copy if rounded else x, y, step)
         copy = rt.empty(*x.shape) if rounded and isinstance(hand_to, RoundedRows) else None
         norm_b.add_normed(y, x, True, copy)
+        return copy
+
+
+@register_part("arrangement", "normed_sum_residual")
+class NormedSumResidual(Arrangement):
+    """x = norm_a(scale x + mixer(x)); x = norm_b(scale x + feed_forward(x)): the norm stands behind the sum of the stream
+    and the sublayer's output, and the sublayers read the stream itself (rounded to the compute dtype for their matrix
+    products); the factor on the stream is the norms' own (Norm.norm_sum).  One kernel forms the sum, normalises it
+    and, on the bfloat16 path, leaves the rounded rows the next sublayer reads; a mixer that gives its output in terms
+    (Mixer.gives_terms) has them normalised and added in the same kernel."""
+    slots = {"mixer": "mixer", "mixer_norm": "norm", "feed_forward": "feed_forward", "feed_forward_norm": "norm"}
+    optional = ("feed_forward", "feed_forward_norm")
+    carries = True
+    _asks = RoundedRows()
+
+    def accepts_carry(self, layer):
+        rt = layer.part("mixer").runtime
+        return self._asks if rt is not None and rt.dtype != torch.float32 else None
+
+    def forward(self, layer, x: torch.Tensor, step, cache: LayerCache, carry=None, hand_to=None):
+        mixer, norm_a = layer.part("mixer"), layer.part("mixer_norm")
+        ff, norm_b = layer.part("feed_forward"), layer.part("feed_forward_norm")
+        rt = mixer.runtime
+        rounded = rt.dtype != torch.float32
+        if not rounded:
+            xin = x
+        elif isinstance(carry, torch.Tensor):
+            xin = carry
+        else:
+            xin = rt.empty(*x.shape)
+            K.cast_rows(x, xin)
+        last = ff is None or norm_b is None
+        y = None
+        if mixer.gives_terms:
+            terms = mixer.terms(xin, step, cache)
+        else:
+            y = rt.empty(*x.shape, dtype=torch.float32)
+            OutputNormResidual._run(mixer, xin, y, step, cache)
+            terms = (Term(y),)
+        hands = rounded and isinstance(hand_to, RoundedRows)
+        copy = rt.empty(*x.shape) if (hands if last else rounded) else None
+        norm_a.norm_sum(x, terms, copy)
+        if last:
+            return copy
+        if y is None:
+            y = rt.empty(*x.shape, dtype=torch.float32)
+        OutputNormResidual._run(ff, copy if rounded else x, y, step)
+        copy = rt.empty(*x.shape) if hands else None
+        norm_b.norm_sum(x, (Term(y),), copy)
         return copy
 
 

@@ -26,12 +26,14 @@ def interleave_rows(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
 
 
 GATE_ACTS = {"silu": K.ACT_NONE, "gelu_erf": K.ACT_GELU_ERF, "gelu_tanh": K.ACT_GELU_TANH, "relu_sq": K.ACT_RELU_SQ}
+CLAMPED = "clamped"          # acts on gate and up together, see SwiGLU
 
 
 @register_part("feed_forward", "swiglu")
 class SwiGLU(FeedForward):
     """A gated feed-forward: Wd (act(Wg xn) * (Wu xn)), act = silu unless `activation` names another ("gelu_tanh",
-    "gelu_erf", "relu_sq").  params: hidden, intermediate, bias, prefix, activation, and the tensors' names gate, up,
+    "gelu_erf", "relu_sq"); or ("clamped", with a `limit` L) Wd (g sigmoid(1.702 g) (u + 1)), g = min(Wg xn, L), u = Wu xn
+    clamped to [-L, L].  params: hidden, intermediate, bias, prefix, activation, limit, and the tensors' names gate, up,
     down (defaults "gate_proj.weight" ... with biases "gate_proj.bias" ...; a name given in full has its bias at
     name + ".b")."""
     replays_prompts = True
@@ -45,9 +47,10 @@ class SwiGLU(FeedForward):
         self.intermediate = int(spec["intermediate"])
         self.bias = bool(spec.get("bias", False))
         act = spec.get("activation", "silu")
-        if act not in GATE_ACTS:
-            raise ValueError(f"gated feed-forward: activation {act!r} is not one of {sorted(GATE_ACTS)}")
-        self.act = GATE_ACTS[act]
+        if act not in GATE_ACTS and act != CLAMPED:
+            raise ValueError(f"gated feed-forward: activation {act!r} is not one of {sorted(GATE_ACTS) + [CLAMPED]}")
+        self.act = K.ACT_CLAMPED_GATE if act == CLAMPED else GATE_ACTS[act]
+        self.limit = float(spec["limit"]) if act == CLAMPED else 0.0
         self.w_names, self.b_names = {}, {}
         for key in ("gate", "up", "down"):
             given = spec.get(key)
@@ -73,7 +76,7 @@ class SwiGLU(FeedForward):
         self.down = Linear(self.runtime, weights[wn["down"]], weights.get(bn["down"]) if self.bias else None)
 
     def forward(self, xn, residual: torch.Tensor, step, emit=None, store: bool = False) -> None:
-        a = self.gate_up(xn, mode=SWIGLU, act=self.act)
+        a = self.gate_up(xn, mode=SWIGLU, act=self.act, limit=self.limit)
         self.down(a, out=residual, mode=STORE_F32 if store else ADD_TO_F32, emit=None if store else emit)
 
 

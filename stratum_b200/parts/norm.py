@@ -3,12 +3,12 @@ RMSNorm: y = x / sqrt(mean(x^2) + eps) * gain  (stratum/native/stratum_arch_llam
 Dynamic Tanh: y = tanh(alpha x) * w + b, elementwise: it stands where a norm would and takes no row statistic."""
 from __future__ import annotations
 
-from typing import Dict, Mapping, Optional
+from typing import Dict, Mapping, Optional, Sequence
 
 import torch
 
 from .. import kernels as K
-from .base import Handover, Norm
+from .base import Handover, Norm, Term
 from .registry import register_part
 from .spec import TensorSpec
 
@@ -72,6 +72,47 @@ class RMSNorm(Norm):
         if head_dim != self.size:
             raise ValueError(f"rmsnorm of size {self.size} asked to normalise heads of {head_dim}")
         K.rmsnorm_heads(x, first_col, n_heads, head_dim, self.gain, self.eps)
+
+
+@register_part("norm", "grouped_rmsnorm")
+class GroupedRMSNorm(Norm):
+    """The row is cut into `groups` equal consecutive parts, each divided by its own root mean square (eps inside the
+    root), and the whole is multiplied by the weight.  One group: the plain RMS norm.
+    params: size, groups, eps, tensor (the weight's whole name) or prefix (then prefix + "weight"), stream (the factor
+    on the residual stream where the norm stands behind the sum of the stream and a sublayer's output; default 1)."""
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        self.size, self.groups = int(spec["size"]), int(spec.get("groups", 1) or 1)
+        if self.size % self.groups:
+            raise ValueError(f"grouped_rmsnorm: {self.size} values do not form {self.groups} equal parts")
+        self.eps, self.stream = float(spec["eps"]), float(spec.get("stream", 1.0))
+        self.tensor = spec.get("tensor")
+        self.gain: Optional[torch.Tensor] = None
+
+    @property
+    def name(self) -> str:
+        return self.tensor or self.prefix + "weight"
+
+    def tensors(self) -> Dict[str, TensorSpec]:
+        return {self.name: TensorSpec((self.size,), role="vector", init="ones")}
+
+    def bind(self, weights: Mapping[str, torch.Tensor]) -> None:
+        self.gain = weights[self.name].contiguous()
+
+    def forward(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        out = self.runtime.empty(x.shape[0] if rows is None else rows.numel(), self.size)
+        K.sum_norm(x, 1.0, (), self.gain, self.groups, self.eps, out, rows=rows)
+        return out
+
+    def norm_sum(self, x: torch.Tensor, terms: Sequence[Term], copy: Optional[torch.Tensor] = None) -> None:
+        K.sum_norm(x, self.stream, terms, self.gain, self.groups, self.eps, x, copy=copy)
+
+    def add_normed(self, y: torch.Tensor, residual: torch.Tensor, accumulate: bool = True,
+                   copy: Optional[torch.Tensor] = None) -> None:
+        if accumulate:
+            raise NotImplementedError("grouped_rmsnorm: no form that adds the normed rows to the stream")
+        K.sum_norm(y, 1.0, (), self.gain, self.groups, self.eps, residual, copy=copy)
 
 
 @register_part("norm", "layernorm")

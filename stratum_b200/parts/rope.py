@@ -27,7 +27,7 @@ from .registry import register_part
 
 def precise_frequencies(rope_dim: int, theta: float, scaling: Optional[dict]) -> (np.ndarray, float):
     """The same table evaluated in float64 and rounded to float32 once, with the rescalings taken as written for any
-    positive factor (linear: inv_k / factor; yarn: the ramp and the magnitude 0.1 ln(factor) + 1)."""
+    positive factor (linear: inv_k / factor; yarn: the ramp and the magnitude 0.1 ln(factor) + 1; llama3: by wavelength)."""
     n_pairs = rope_dim // 2
     k = np.arange(n_pairs, dtype=np.float64)
     base = float(theta) ** (-2.0 * k / float(rope_dim))
@@ -47,6 +47,13 @@ def precise_frequencies(rope_dim: int, theta: float, scaling: Optional[dict]) ->
         hi = min(math.ceil(corr(float(scaling.get("beta_slow", 1.0)))), rope_dim - 1)
         ramp = np.clip((k - lo) / max(hi - lo, 0.001), 0.0, 1.0)
         return (base / factor * ramp + base * (1.0 - ramp)).astype(np.float32), 0.1 * math.log(factor) + 1.0
+    if kind == "llama3":
+        low, high = float(scaling["low_freq_factor"]), float(scaling["high_freq_factor"])
+        orig = float(scaling["original_max_position"])
+        wave = 2.0 * math.pi / base
+        s = (orig / wave - low) / (high - low) if high != low else np.zeros_like(base)       # (no wavelength lies between)
+        mixed = (1.0 - s) * base / factor + s * base
+        return np.where(wave < orig / high, base, np.where(wave > orig / low, base / factor, mixed)).astype(np.float32), 1.0
     raise ValueError(f"rope scaling kind {kind!r} has no precise form")
 
 

@@ -1,4 +1,5 @@
-"""Grouped-query attention over a sliding window, with normalised queries and keys and a sink in the softmax.
+"""Grouped-query attention over a sliding window or over chunks, with normalised queries and keys and, optionally, a
+sink in the softmax, a factor per head on the scores and a gate on the output.
 
 Per token, with h the mixer's input and p its position:  q = Wq h ([heads][d]), k = Wk h ([kv heads][d]); v = k as
 projected (no value matrix), or (`v_dim`) v = Wv h ([kv heads][dv]); the projections may have biases.  q and k are
@@ -8,13 +9,15 @@ heads; then the first dimensions of every head are rotated by the position encod
 (2i, 2i + 1) or in pairs (i, i + n/2) as the encoding says.  Head j (kv head j / (heads / kv heads)):
 
     s_t = (q_j . k_t) * scale         for the keys t with 0 <= p - t < window or t < keep_first (window 0: every t <= p)
+                                      and, with chunks of C positions, floor(t / C) = floor(p / C); times temp_j where
+                                      the mixer has a factor per head
     a_t = exp(s_t) / (sum_t exp(s_t) + exp(sink_j))            (the sink has no key and no value and is not scaled)
-    o_j = sum_t a_t v_t;      result = Wo concat_j(o_j)
+    o_j = sum_t a_t v_t;      result = Wo concat_j(o_j)         (with an output gate: concat_j(o_j) * sigmoid(Wg h))
 
 The sink is a learned number per head, the constant 0 (`sink: "zero"`: one added to every denominator), or absent.
 The projections run as one product whose float32 sums go to one kernel that normalises, rotates, rounds once and
 appends to the cache (csrc/qk_norm_rope.cu); the attention itself is the general kernel (kernels.AttentionShape) with
-its window, kept first keys and sink parameters.
+its window, chunk, kept first keys, sink and gate parameters.
 """
 from __future__ import annotations
 
@@ -38,9 +41,11 @@ class SinkAttention(Mixer):
     positions below it stay visible), eps (of the two norms), position (PartSpec of a rotating position encoding, or
     None), sink (True: a learned number per head, the default; "zero": the constant 0; False: none), v_dim (None:
     the values are the keys as projected; else a value matrix of n_kv_heads * v_dim rows), qk_norm ("whole", the
-    default, or "per_head"), bias (biases on the projections: name + ".b"), prefix, and the tensor names q, k, v, o,
-    q_norm, k_norm, sink (defaults: q, k, v, o, q.norm, k.norm, sink)."""
+    default, or "per_head"), bias (biases on the projections: name + ".b"), chunk (0: none), temp (True: a learned factor
+    per head on the scores), gate (True: an output gate per element, with a matrix of n_heads * dv rows), prefix, and the
+    tensor names q, k, v, o, q_norm, k_norm, sink, temp, g (defaults: q, k, v, o, q.norm, k.norm, sink, temp, g)."""
     stores_output = True
+    splits_projection = True
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
@@ -51,6 +56,8 @@ class SinkAttention(Mixer):
         self.scale, self.eps = float(spec["scale"]), float(spec["eps"])
         self.window = int(spec.get("window", 0) or 0)
         self.keep_first = int(spec.get("keep_first", 0) or 0) if self.window else 0
+        self.chunk = int(spec.get("chunk", 0) or 0)
+        self.has_temp, self.has_gate = bool(spec.get("temp", False)), bool(spec.get("gate", False))
         sink = spec.get("sink", True)
         if sink not in (True, False, "zero"):
             raise ValueError(f"sink_attention: sink {sink!r} is not one of True, False, 'zero'")
@@ -71,21 +78,23 @@ class SinkAttention(Mixer):
             if layout is None or 2 * layout[0] > self.d:
                 raise ValueError("sink_attention rotates pairs among a head's first dimensions")
             self.half = not layout[1]
-        defaults = {"q": "q", "k": "k", "v": "v", "o": "o", "q_norm": "q.norm", "k_norm": "k.norm", "sink": "sink"}
+        defaults = {"q": "q", "k": "k", "v": "v", "o": "o", "q_norm": "q.norm", "k_norm": "k.norm", "sink": "sink",
+                    "temp": "temp", "g": "g"}
         self.names = {k: self.prefix + str(spec.get(k + "_tensor", v)) for k, v in defaults.items()}
         self.q_cols, self.k_cols = self.n_heads * self.d, self.n_kv * self.d
         self.v_cols = self.n_kv * self.dv if self.own_values else 0
         self.o_cols = self.n_heads * self.dv
+        self.width = self.q_cols + self.k_cols + self.v_cols + (self.o_cols if self.has_gate else 0)
         self.w_in: Optional[Linear] = None
         self.w_o: Optional[Linear] = None
         self.shape: Optional[K.AttentionShape] = None
 
     def _stacked(self):
-        return ("q", "k", "v") if self.own_values else ("q", "k")
+        return ("q", "k") + (("v",) if self.own_values else ()) + (("g",) if self.has_gate else ())
 
     def tensors(self) -> Dict[str, TensorSpec]:
         n = self.names
-        cols = {"q": self.q_cols, "k": self.k_cols, "v": self.v_cols}
+        cols = {"q": self.q_cols, "k": self.k_cols, "v": self.v_cols, "g": self.o_cols}
         t = {n[key]: TensorSpec((cols[key], self.hidden)) for key in self._stacked()}
         if self.bias:
             t.update({n[key] + ".b": TensorSpec((cols[key],), role="vector") for key in self._stacked()})
@@ -94,12 +103,19 @@ class SinkAttention(Mixer):
         t[n["k_norm"]] = TensorSpec((self.d if self.per_head else self.k_cols,), role="vector", init="ones")
         if self.has_sink:
             t[n["sink"]] = TensorSpec((self.n_heads,), role="vector", init="zeros")
+        if self.has_temp:
+            t[n["temp"]] = TensorSpec((self.n_heads,), role="vector", init="ones")
         return t
 
-    def bind(self, weights: Mapping[str, torch.Tensor]) -> None:
+    def input_weights(self, weights: Mapping[str, torch.Tensor]):
         n = self.names
         b = torch.cat([weights[n[key] + ".b"] for key in self._stacked()]).contiguous() if self.bias else None
-        self.w_in = Linear(self.runtime, torch.cat([weights[n[key]] for key in self._stacked()], dim=0).contiguous(), b)
+        return torch.cat([weights[n[key]] for key in self._stacked()], dim=0).contiguous(), b
+
+    def bind(self, weights: Mapping[str, torch.Tensor], own_projection: bool = True) -> None:
+        n = self.names
+        if own_projection:
+            self.w_in = Linear(self.runtime, *self.input_weights(weights))
         self.w_o = Linear(self.runtime, weights[n["o"]])
         self.q_gain, self.k_gain = weights[n["q_norm"]].contiguous(), weights[n["k_norm"]].contiguous()
         self.sink = None
@@ -108,20 +124,21 @@ class SinkAttention(Mixer):
         elif self.zero_sink:
             self.sink = torch.zeros(self.n_heads, dtype=torch.float32, device=self.q_gain.device)
         self.shape = K.AttentionShape(self.n_heads, self.n_heads // self.n_kv, 1, self.d, self.dv, False, self.scale,
-                                      window=self.window, sink=self.sink, keep_first=self.keep_first)
+                                      window=self.window, sink=self.sink, keep_first=self.keep_first, chunk=self.chunk,
+                                      head_scale=weights[n["temp"]].contiguous() if self.has_temp else None)
 
     def cache_spec(self) -> KVSpec:
         order = "normed_rotated" + ("_half" if self.half else "") + ("" if self.own_values else "_values_raw")
         if not self.own_values:
-            return KVSpec(self.n_kv, self.d, self.window, order, keep_first=self.keep_first)
+            return KVSpec(self.n_kv, self.d, self.window, order, keep_first=self.keep_first, chunk=self.chunk)
         return KVSpec(self.n_kv, self.d, self.window, order, value_heads=self.n_kv, value_dim=self.dv,
-                      keep_first=self.keep_first)
+                      keep_first=self.keep_first, chunk=self.chunk)
 
-    def forward(self, xin, residual: torch.Tensor, step, cache: LayerCache, store: bool = False) -> None:
+    def forward(self, xin, residual: torch.Tensor, step, cache: LayerCache, store: bool = False, proj=None) -> None:
         T = xin.shape[0]
-        width = self.q_cols + self.k_cols + self.v_cols
-        proj = self.runtime.empty(T, padded(width), dtype=torch.float32)
-        self.w_in(xin, out=proj[:, :width], mode=STORE_F32)
+        if proj is None:
+            proj = self.runtime.empty(T, padded(self.width), dtype=torch.float32)[:, :self.width]
+            self.w_in(xin, out=proj, mode=STORE_F32)
         q = self.runtime.empty(T, padded(self.q_cols))
         rot = self.position.rotary() if self.position is not None else None
         K.qk_norm_rope(proj, step.token_pos, step.token_seq, cache.block_table, self.q_gain, self.k_gain,
@@ -130,5 +147,6 @@ class SinkAttention(Mixer):
                        per_head=self.per_head, half=self.half, magnitude=1.0 if rot is None else rot.magnitude)
         out = self.runtime.empty(T, padded(self.o_cols))
         from . import attention_dispatch
-        attention_dispatch.run_general(self, self.shape, q, cache, step, out)
+        gate = proj[:, self.width - self.o_cols:] if self.has_gate else None
+        attention_dispatch.run_general(self, self.shape, q, cache, step, out, gate)
         self.w_o(out[:, :self.o_cols], out=residual, mode=STORE_F32 if store else ADD_TO_F32)
