@@ -42,8 +42,11 @@ __device__ __forceinline__ void sn_axpy(float4& z, float a, float4 y, float4 g) 
 }
 
 // Rows whose groups are a multiple of four values, at most KEEP pieces of four per thread; `team` warps per group.
+// (as many warps as the registers of KEEP pieces leave room for)
+__host__ __device__ constexpr int sn_most_warps(int keep) { return keep == 2 ? 32 : (keep == 4 ? 24 : 16); }
+
 template <typename T, int KEEP>
-__global__ void sum_norm_vec_kernel(const SumNorm P, int team) {
+__global__ void __launch_bounds__(sn_most_warps(KEEP) * 32) sum_norm_vec_kernel(const SumNorm P, int team) {
   __shared__ float part[SN_TERMS][32], zpart[32];
   pdl_trigger();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
@@ -173,11 +176,11 @@ static int launch_sum_norm(const SumNorm& P, cudaStream_t stream) {
   for (int j = 0; j < SN_TERMS; j++) bits |= (uintptr_t)P.y[j] | (uintptr_t)P.y_gain[j];
   // (the choice depends on the row's length and on alignment alone, which a model's buffers share from step to step)
   if (size % 4 == 0 && (bits & 15) == 0 && n_groups <= 32) {
-    const int pieces = size / 4, most = 32 / n_groups;
+    const int pieces = size / 4;
     int keep = 0, team = 0;
     for (int k = 2; k <= 8 && !keep; k *= 2) {
       team = (pieces + 32 * k - 1) / (32 * k);
-      if (team <= most) keep = k;
+      if (team * n_groups <= sn_most_warps(k)) keep = k;
     }
     if (keep) {
       const dim3 block(n_groups * team * 32);

@@ -1258,7 +1258,7 @@ class LinearRecurrence:
                         ("seq_slot", step.seq_slot)):
             _need(t, name, torch.int32)
         W, T = self.width, proj.shape[0]
-        if proj.shape[1] < 2 * W or out.shape[0] != T or out.shape[1] < W or state.shape[1] < (1 + self.taps) * W:
+        if proj.shape[1] < 2 * W or out.shape[0] != T or step.token_seq.numel() != T or out.shape[1] < W or state.shape[1] < (1 + self.taps) * W:
             raise KernelError("linear recurrence: buffers and sizes disagree")
         p = _Lru()
         p.y, p.x = proj.data_ptr(), proj.data_ptr() + 4 * W
