@@ -7,6 +7,7 @@
     python bench.py --compare dabodra       # the same for the Dabodra decoder
     python bench.py --compare vitinex       # the Vitinex decoder beside the Dabodra and the Llama decoder of equal size
     python bench.py --compare mokatar       # the Mokatar decoder beside the same two
+    python bench.py --compare getizen       # the Getizen decoder beside the Mokatar and the Llama decoder of equal size
 
 Prints ONE JSON line.  `value` is decoded tokens per second at the given batch, with every
 sequence's cache filled to the given context at the end of the timed steps (so the timed steps
@@ -179,6 +180,34 @@ def mokatar_config(size, n_layers):
         "layers": layers, "loop": {"start": 0, "stop": n_layers, "times": 1}})
 
 
+# --compare getizen: the same widths, heads and vocabulary, beside the Mokatar decoder (the closest one here: attention
+# that is cut off behind the same 1,024 positions, linear attention with the same state of 128 x 128 per head) and the
+# Llama decoder.  Three layers of chunked attention and a linear recurrence side by side (as many channels as the model
+# is wide, in blocks of 256) to one layer of retention; the dense feed-forwards hold as many weights as the Llama
+# decoder's.
+GETIZEN_SIZES = {
+    "1b": {"dim": 128, "vdim": 128, "chunk": 1024, "block": 256, "ret_dim": 128, "ret_vdim": 128},
+    "8b": {"dim": 128, "vdim": 128, "chunk": 1024, "block": 256, "ret_dim": 128, "ret_vdim": 128},
+}
+
+
+def getizen_config(size, n_layers):
+    from stratum_b200.config import GetizenConfig
+    z, g = COMPARE_SIZES[size], GETIZEN_SIZES[size]
+    left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": g["dim"], "vdim": g["vdim"], "scale": g["dim"] ** -0.5,
+            "mask": {"size": g["chunk"]},
+            "rot": {"base": 10000.0, "dims": g["dim"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    right = {"width": z["width"], "blocks": z["width"] // g["block"], "conv": 4}
+    ret = {"heads": z["heads"], "dim": g["ret_dim"], "vdim": g["ret_vdim"],
+           "decay": [1.0 - 2.0 ** (-5 - 5 * h / z["heads"]) for h in range(z["heads"])],
+           "rot": {"base": 10000.0, "dims": g["ret_dim"]}}
+    mlp = {"kind": "dense", "ff": z["llama_inner"], "limit": 7.0}
+    layers = [{"type": "retention", "mixer": ret, "mlp": mlp} if i % 4 == 3 else
+              {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": mlp} for i in range(n_layers)]
+    return GetizenConfig.from_dict({"architecture": "Getizen", "vocab": z["vocab"], "width": z["width"],
+                                    "norm": {"eps": 1e-5, "groups": 2}, "postln_alpha": 1.5, "layers": layers})
+
+
 def llama_like(size, n_layers):
     from stratum_b200.config import LlamaConfig
     z = COMPARE_SIZES[size]
@@ -218,8 +247,8 @@ def kernel_times(llm, batch, context, prefill_tokens, vocab, rng):
 
 
 def compare_models(args, rng):
-    """Prefill and decode throughput of the Nibelorn, the Dabodra, the Vitinex or the Mokatar decoder beside a Llama
-    decoder of equal size (the Vitinex and the Mokatar decoder also beside the Dabodra decoder): one
+    """Prefill and decode throughput of the Nibelorn, the Dabodra, the Vitinex, the Mokatar or the Getizen decoder beside
+    a Llama decoder of equal size (Vitinex and Mokatar also beside the Dabodra, Getizen beside the Mokatar decoder): one
     prompt of --prefill-tokens, and decode steps of --batch sequences at --context tokens (random bf16 weights,
     device-timed as the main workload is); with --kernels also the device time of every kernel of one prompt and one
     decode step.  One JSON line."""
@@ -228,8 +257,9 @@ def compare_models(args, rng):
     n_layers = args.layers or 8
     which = args.compare
     make = {"nibelorn": nibelorn_config, "dabodra": dabodra_config, "vitinex": vitinex_config,
-            "mokatar": mokatar_config}[which]
-    others = [("llama", llama_like)] + ([("dabodra", dabodra_config)] if which in ("vitinex", "mokatar") else [])
+            "mokatar": mokatar_config, "getizen": getizen_config}[which]
+    others = [("llama", llama_like)] + ([("dabodra", dabodra_config)] if which in ("vitinex", "mokatar") else []) \
+        + ([("mokatar", mokatar_config)] if which == "getizen" else [])
     out = {"compare": which, "layers": n_layers, "batch": args.batch, "context": args.context,
            "prefill_tokens": args.prefill_tokens, "dtype": "bf16", "data": "synthetic: random-init weights",
            "sizes": {}}
@@ -487,9 +517,9 @@ def main() -> int:
                     help="prompt length of --prefill-only (the default JSON line always uses 2,048)")
     ap.add_argument("--shape", default="llama3.1-8b", choices=["llama3.1-8b"] + sorted(OTHER_SHAPES),
                     help="layer sizes for the short lines of --decode-only / --prefill-only")
-    ap.add_argument("--compare", default=None, choices=["nibelorn", "dabodra", "vitinex", "mokatar"],
+    ap.add_argument("--compare", default=None, choices=["nibelorn", "dabodra", "vitinex", "mokatar", "getizen"],
                     help="instead of the main workload: prefill and decode throughput of the Nibelorn, the Dabodra, "
-                         "the Vitinex or the Mokatar decoder beside a Llama decoder of equal size (Vitinex and Mokatar also beside Dabodra), at 1B-like and 8B-like layer sizes (--layers of "
+                         "the Vitinex or the Mokatar decoder beside a Llama decoder of equal size (Vitinex and Mokatar also beside Dabodra, Getizen beside Mokatar), at 1B-like and 8B-like layer sizes (--layers of "
                          "them, default 8)")
     ap.add_argument("--kernels", action="store_true",
                     help="with --compare: also the device time of every kernel of one prompt and one decode step")
