@@ -31,6 +31,11 @@
 // V is used as stored, [key][dim]: as the B operand of P V its n index (dim) is the contiguous one
 // ("MN-major"), which the instruction takes directly; no transpose is made anywhere.
 //
+// SPLIT: the probabilities stay as wide as two bfloat16 (p = hi + lo to 16 bits of mantissa): P has a second buffer, and
+// O += P_hi V + P_lo V.  For mixers whose attention weights are not to be rounded to bfloat16.  This form also knows
+// chunks (with `chunk` > 0 a position sees only keys of its own chunk of that many positions) and an output gate (where
+// pre-activations are given, o is multiplied by sigmoid(gate) element by element before it is stored).
+//
 // Every mbarrier wait is bounded (see gemm_tc.cu): on expiry a code goes to the status word and the CTA winds
 // down, freeing its tensor memory.
 #include <math.h>
@@ -49,16 +54,26 @@ struct FaParams {
   const int* qb_seq; const int* qb_tok0; const int* qb_ntok;
   bf16* out; int ldo;
   int* status;
-  int n_q, n_kv, gs, tokens_per_tile, window;
+  const float* gate; int ld_gate;
+  int n_q, n_kv, gs, tokens_per_tile, window, chunk;
   float scale_log2;        // scale * log2(e): exponentials are taken with exp2
 };
 
-template <int HD, int NH>
+// the first key a position sees
+template <bool CHUNKS>
+__device__ __forceinline__ int fa_first_key(const FaParams& P, int pos) {
+  int lo = (P.window > 0 && pos - P.window + 1 > 0) ? pos - P.window + 1 : 0;
+  if (CHUNKS && P.chunk > 0) lo = max(lo, pos - pos % P.chunk);
+  return lo;
+}
+
+template <int HD, int NH, bool SPLIT>
 struct FaSmem {
   alignas(1024) bf16 q[NH][FA_ROWS * HD];             // per half: [HD/64 blocks of 64 dims][128 rows][64]
   alignas(1024) bf16 k[FA_STAGES][FA_KEYS * HD];      // [HD/64][64 keys][64 dims]
   alignas(1024) bf16 v[FA_STAGES][FA_KEYS * HD];      // [HD/64][64 keys][64 dims]
   alignas(1024) bf16 p[NH][FA_ROWS * FA_KEYS];        // per half: [128 rows][64 keys]; at the end: the rows' two half sums
+  alignas(1024) bf16 p_lo[SPLIT ? NH : 1][SPLIT ? FA_ROWS * FA_KEYS : 8];     // SPLIT: the low parts, laid out alike
   uint64_t q_full, k_full[FA_STAGES], v_full[FA_STAGES];
   uint64_t s_full[NH][2], p_full[NH], pv_full[NH][2];
   uint32_t tmem_base;
@@ -93,12 +108,12 @@ __device__ __forceinline__ FaHalf fa_half(const FaParams& P, int h, int seq, int
   return H;
 }
 
-template <int HD, int NH>
+template <int HD, int NH, bool SPLIT>
 __global__ void __launch_bounds__(FA_THREADS(NH), NH == 1 ? 2 : 1)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, const FaParams P) {
   extern __shared__ __align__(1024) uint8_t smem_raw[];
-  using Smem = FaSmem<HD, NH>;
+  using Smem = FaSmem<HD, NH, SPLIT>;
   Smem& S = *reinterpret_cast<Smem*>(smem_raw);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   constexpr int DB = HD / 64;                           // blocks of 64 dims
@@ -143,7 +158,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 
   // keys are walked from the first half's first tile (a later half whose window begins further on masks them out)
   const int first_pos = P.token_pos[tok0];
-  const int lo_tile = (P.window > 0 && first_pos - P.window + 1 > 0) ? (first_pos - P.window + 1) / FA_KEYS : 0;
+  const int lo_tile = fa_first_key<SPLIT>(P, first_pos) / FA_KEYS;
   const int nt0 = fa_half(P, 0, seq, first_pos, ntok, lo_tile).n_tiles;
   const int nt1 = NH > 1 ? fa_half(P, 1, seq, first_pos, ntok, lo_tile).n_tiles : 0;      // (never more than nt0 + 1)
   const int n_tiles_max = max(nt0, nt1);
@@ -223,7 +238,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       const uint32_t tmem_h = tmem_base + h * 256;
       bool ok = __all_sync(0xffffffffu, mbar_wait(&S.q_full, 0, abort_flag));
       if (!ok && lane == 0) FA_FAIL(202);
-      const uint32_t q_addr = smem_u32(S.q[h]), p_addr = smem_u32(S.p[h]);
+      const uint32_t q_addr = smem_u32(S.q[h]), p_addr = smem_u32(S.p[h]), p_lo_addr = smem_u32(S.p_lo[SPLIT ? h : 0]);
       auto issue_scores = [&](int j) -> bool {
         const int s = j % FA_STAGES, b = j & 1;
         if (!__all_sync(0xffffffffu, mbar_wait(&S.k_full[s], (j / FA_STAGES) & 1, abort_flag))) {
@@ -257,6 +272,12 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           for (int kk = 0; kk < 4; kk++)        // 16 keys a step: 32 bytes along a row of P, 16 rows of V
             umma_bf16(tmem_h + COL_PV, smem_desc_sw128(p_addr + kk * 32),
                       smem_desc_sw128_mn(v_addr + kk * 16 * 128, FA_KEYS * 128), idesc_pv, (j | kk) ? 1u : 0u);
+          if (SPLIT) {
+#pragma unroll
+            for (int kk = 0; kk < 4; kk++)
+              umma_bf16(tmem_h + COL_PV, smem_desc_sw128(p_lo_addr + kk * 32),
+                        smem_desc_sw128_mn(v_addr + kk * 16 * 128, FA_KEYS * 128), idesc_pv, 1u);
+          }
           umma_commit(&S.pv_full[h][j & 1]);    // to the softmax warps (P is read, O has the tile), and to the
                                                 // producer: V of this tile is read
         }
@@ -276,7 +297,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int tok = row / P.gs, head = row % P.gs;
     const bool valid = tok < H.ntok;
     const int pos = H.first_pos + (valid ? tok : 0);
-    const int lo = (P.window > 0 && pos - P.window + 1 > 0) ? pos - P.window + 1 : 0;
+    const int lo = fa_first_key<SPLIT>(P, pos), lo_last = SPLIT ? fa_first_key<SPLIT>(P, H.last_pos) : 0;
     const uint32_t lane_addr = tmem_base + h * 256 + ((uint32_t)(quarter * 32) << 16);
     constexpr int OD = HD / 2;                           // output dims per thread
     const uint32_t o_addr = lane_addr + COL_PV + half * OD;
@@ -298,7 +319,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       // maximum over the whole tile; keys beyond a row's own position (or before its window) are masked, which
       // only tiles on the diagonal (or at the window's edge) need
       const int key0 = (lo_tile + j) * FA_KEYS;
-      const bool needs_mask = (key0 + FA_KEYS - 1 > H.first_pos) || (P.window > 0) || (H.ntok < P.tokens_per_tile);
+      const bool needs_mask = (key0 + FA_KEYS - 1 > H.first_pos) || (SPLIT ? key0 < lo_last : P.window > 0) || (H.ntok < P.tokens_per_tile);
       // (four running maxima, then combined: one chain of 64 dependent comparisons would cost more time than
       // everything else a thread does per tile)
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -323,7 +344,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       if (grow) m_ref = tile_max;
       const float m_use = (m_ref == -INFINITY) ? 0.f : m_ref;
       // probabilities exp2(s * scale - ref) of this thread's keys, their sum, and P in the layout the MMA reads
-      uint32_t packed[16];
+      uint32_t packed[16], packed_lo[SPLIT ? 16 : 1];
       float sum0 = 0.f, sum1 = 0.f;
 #pragma unroll
       for (int i = 0; i < 32; i += 2) {
@@ -335,8 +356,15 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         // shortened values, so the common part of that factor divides out and what stays is as wide as
         // round-to-nearest's error.
         const uint32_t u = __byte_perm(__float_as_uint(p0), __float_as_uint(p1), 0x7632);
-        sum0 += __uint_as_float(u << 16);
-        sum1 += __uint_as_float(u & 0xffff0000u);
+        if (SPLIT) {                           // the rest of every probability, shortened likewise: 16 bits together
+          const float r0 = p0 - __uint_as_float(u << 16), r1 = p1 - __uint_as_float(u & 0xffff0000u);
+          packed_lo[i >> 1] = __byte_perm(__float_as_uint(r0), __float_as_uint(r1), 0x7632);
+          sum0 += p0;
+          sum1 += p1;
+        } else {
+          sum0 += __uint_as_float(u << 16);
+          sum1 += __uint_as_float(u & 0xffff0000u);
+        }
         packed[i >> 1] = u;
       }
       if (j > 0) {
@@ -368,6 +396,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           const int chunk = half * 4 + c;                // 16-byte chunk = 8 keys
           *reinterpret_cast<uint4*>(prow + ((chunk ^ (row & 7)) << 4)) =
               make_uint4(packed[4 * c], packed[4 * c + 1], packed[4 * c + 2], packed[4 * c + 3]);
+          if (SPLIT)
+            *reinterpret_cast<uint4*>(reinterpret_cast<uint8_t*>(S.p_lo[h]) + row * 128 + ((chunk ^ (row & 7)) << 4)) =
+                make_uint4(packed_lo[4 * c], packed_lo[4 * c + 1], packed_lo[4 * c + 2], packed_lo[4 * c + 3]);
         }
       }
       fence_async_shared();
@@ -390,12 +421,26 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       const float inv = 1.0f / (l_buf[row] + l_buf[FA_ROWS + row]);
       bf16* op = P.out + (size_t)(tok0 + h * P.tokens_per_tile + (valid ? tok : 0)) * P.ldo +
                  (size_t)(kvh * P.gs + head) * HD + half * OD;
+      const float* gp = nullptr;
+      if (SPLIT && P.gate) {
+        pdl_wait();                                      // (the gate comes from an earlier kernel: this thread waits too)
+        gp = P.gate + (size_t)(tok0 + h * P.tokens_per_tile + (valid ? tok : 0)) * P.ld_gate +
+             (size_t)(kvh * P.gs + head) * HD + half * OD;
+      }
 #pragma unroll
       for (int c = 0; c < OD; c += 32) {
         float o[32];
         tmem_ld32f(o_addr + c, o);                       // (all lanes take part in the load; only valid rows store)
         tmem_ld_wait();
         if (valid) {
+          if (SPLIT && gp) {
+#pragma unroll
+            for (int i = 0; i < 32; i += 4) {
+              const float4 z = ld_fresh(reinterpret_cast<const float4*>(gp + c + i));
+              o[i] = __fdividef(o[i], 1.0f + __expf(-z.x)); o[i + 1] = __fdividef(o[i + 1], 1.0f + __expf(-z.y));
+              o[i + 2] = __fdividef(o[i + 2], 1.0f + __expf(-z.z)); o[i + 3] = __fdividef(o[i + 3], 1.0f + __expf(-z.w));
+            }
+          }
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
             uint4 w;
@@ -432,11 +477,11 @@ static int make_map_nd(CUtensorMap* map, const void* base, int rank, const cuuin
   return r == CUDA_SUCCESS ? 0 : STRATUM_ERR_SHAPE;
 }
 
-template <int HD, int NH>
+template <int HD, int NH, bool SPLIT>
 static int launch_attention_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const FaParams& P,
                                int n_qblocks, cudaStream_t stream) {
-  const size_t smem = sizeof(FaSmem<HD, NH>);
-  auto kern = attention_tc_kernel<HD, NH>;
+  const size_t smem = sizeof(FaSmem<HD, NH, SPLIT>);
+  auto kern = attention_tc_kernel<HD, NH, SPLIT>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -449,16 +494,20 @@ static int launch_attention_tc(const CUtensorMap& mq, const CUtensorMap& mk, con
 // q: bf16 [tokens][ldq], query heads first (n_q * head_dim values per row are used).
 // k_cache / v_cache: bf16 [n_pages][n_kv][64][head_dim].  Query tiles (qb_*): runs of at most
 // halves * 128 / (n_q / n_kv) consecutive new tokens of one sequence (halves: 1 or 2, see the top of this file).
-// head_dim 64 or 128; 128 % (n_q / n_kv) == 0; pages of 64 tokens.
+// head_dim 64 or 128; 128 % (n_q / n_kv) == 0; pages of 64 tokens.  split, chunk, gate (float32 [tokens][ld_gate], n_q *
+// head_dim columns, or null): see the top of this file; split goes with halves = 2.
 STRATUM_EXPORT int stratum_attention_tc(const void* q, int ldq, const void* k_cache, const void* v_cache,
                                         long long n_pages, const int* token_pos, const int* block_table,
                                         int bt_stride, const int* qb_seq, const int* qb_tok0, const int* qb_ntok,
                                         int n_qblocks, void* out, int ldo, int n_tokens, int n_q, int n_kv,
-                                        int head_dim, int page_tokens, int window, float scale, int halves,
-                                        int* status, cudaStream_t stream) {
+                                        int head_dim, int page_tokens, int window, float scale, int halves, int split,
+                                        int chunk, const float* gate, int ld_gate, int* status, cudaStream_t stream) {
   if (n_tokens <= 0 || n_qblocks <= 0) return 0;
   if (halves != 1 && halves != 2) return STRATUM_ERR_SHAPE;
   if (head_dim != 64 && head_dim != 128) return STRATUM_ERR_SHAPE;
+  if (chunk < 0 || window < 0 || (split && halves != 2) || !(scale > 0.f)) return STRATUM_ERR_SHAPE;
+  if ((gate || chunk) && !split) return STRATUM_ERR_SHAPE;
+  if (gate && (ld_gate < n_q * head_dim || ld_gate % 4 != 0 || ((uintptr_t)gate & 15) != 0)) return STRATUM_ERR_ALIGN;
   if (n_kv < 1 || n_q % n_kv != 0 || page_tokens != FA_KEYS) return STRATUM_ERR_SHAPE;
   const int gs = n_q / n_kv;
   if (gs > FA_ROWS || FA_ROWS % gs != 0) return STRATUM_ERR_SHAPE;
@@ -486,11 +535,16 @@ STRATUM_EXPORT int stratum_attention_tc(const void* q, int ldq, const void* k_ca
   P.qb_seq = qb_seq; P.qb_tok0 = qb_tok0; P.qb_ntok = qb_ntok;
   P.out = (bf16*)out; P.ldo = ldo; P.status = status;
   P.n_q = n_q; P.n_kv = n_kv; P.gs = gs; P.tokens_per_tile = R; P.window = window;
+  P.chunk = chunk; P.gate = gate; P.ld_gate = ld_gate;
   P.scale_log2 = scale * 1.4426950408889634f;
-  if (halves == 2) {
-    if (head_dim == 64) return launch_attention_tc<64, 2>(mq, mk, mv, P, n_qblocks, stream);
-    return launch_attention_tc<128, 2>(mq, mk, mv, P, n_qblocks, stream);
+  if (split) {
+    if (head_dim == 64) return launch_attention_tc<64, 2, true>(mq, mk, mv, P, n_qblocks, stream);
+    return launch_attention_tc<128, 2, true>(mq, mk, mv, P, n_qblocks, stream);
   }
-  if (head_dim == 64) return launch_attention_tc<64, 1>(mq, mk, mv, P, n_qblocks, stream);
-  return launch_attention_tc<128, 1>(mq, mk, mv, P, n_qblocks, stream);
+  if (halves == 2) {
+    if (head_dim == 64) return launch_attention_tc<64, 2, false>(mq, mk, mv, P, n_qblocks, stream);
+    return launch_attention_tc<128, 2, false>(mq, mk, mv, P, n_qblocks, stream);
+  }
+  if (head_dim == 64) return launch_attention_tc<64, 1, false>(mq, mk, mv, P, n_qblocks, stream);
+  return launch_attention_tc<128, 1, false>(mq, mk, mv, P, n_qblocks, stream);
 }

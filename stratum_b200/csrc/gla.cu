@@ -23,24 +23,7 @@
 #include <math.h>
 
 #include "common.cuh"
-
-struct Gla {
-  const float* proj;        // [tokens][ld]
-  void* inner;              // [tokens][ld_inner], the compute dtype: the decay's inner projection (cast)
-  const float* head_decay;  // [n_heads] or null: the decays are alpha's
-  const float* gain;        // [vdim] or null: none
-  float* alpha;             // [tokens][n_heads * dim]: z when `decay` begins, alpha when it ends
-  float* o_raw;             // [tokens][n_heads * vdim]
-  void* out;                // [tokens][ldo] compute dtype
-  float* state;             // [slots][state_stride]: S^T [n_heads][vdim][dim]
-  const int* token_seq;
-  const int* seq_start;     // [seqs + 1]
-  const int* seq_slot;      // [seqs]
-  int ld, ldo, n_tokens, n_seqs;
-  int n_heads, dim, vdim, rank;
-  int state_stride, write_state, ld_inner, rot_pairs;
-  float eps, inv_tau, q_scale, reserved;
-};
+#include "gla.h"
 
 __device__ __forceinline__ float gla_silu(float z) { return z / (1.0f + expf(-z)); }
 
@@ -89,7 +72,6 @@ __global__ void __launch_bounds__(256) gla_rotate_kernel(const Gla P, const floa
 
 // ---------------------------------------------------------------- the recurrence
 #define GLA_THREADS 128
-#define GLA_ROWS 16           // rows of a column of S that a lane holds
 #define GLA_MAX_CHUNK 16      // tokens staged in shared memory at a time, at most
 
 __device__ __forceinline__ void gla_copy4(float* dst_shared, const float* src) {
@@ -253,16 +235,6 @@ __global__ void __launch_bounds__(128) gla_finish_kernel(const Gla P) {
   const float mul = 1.0f / sqrtf(ss / (float)V + P.eps);
   for (int d = lane; d < V; d += 32)
     out[d] = from_float<T>(ld_fresh(o + d) * mul * (P.gain ? P.gain[d] : 1.0f) * gla_silu(ld_fresh(g + d)));
-}
-
-static int gla_check(const Gla& P) {
-  if (P.n_heads < 1 || P.dim < 1 || P.vdim < 1 || P.rank < (P.head_decay ? 0 : 1)) return STRATUM_ERR_SHAPE;
-  if (P.ld < 2 * P.n_heads * P.dim + 2 * P.n_heads * P.vdim + P.rank || P.ldo < P.n_heads * P.vdim)
-    return STRATUM_ERR_SHAPE;
-  if (P.state_stride < P.n_heads * P.dim * P.vdim) return STRATUM_ERR_SHAPE;
-  if (P.dim > 32 * GLA_ROWS) return STRATUM_ERR_LIMIT;
-  if (P.n_heads > 65535 || P.n_seqs > 65535) return STRATUM_ERR_LIMIT;
-  return 0;
 }
 
 static unsigned gla_blocks(size_t n) {

@@ -3,7 +3,7 @@
 // Per token, from the float32 sums of the input projection (branches y and x, `width` columns each):
 //   u = conv_b + sum_j conv_w[j] x(t - taps + 1 + j)          per channel, inputs before the sequence's start are zero
 //   r, i = sigmoid(A_b u_b + .), sigmoid(B_b u_b + .)         per block b of `size` neighbouring channels
-//   a = exp(rate * r);  S <- a S + sqrt(1 - a^2) i u          1 - a^2 taken as -expm1(2 rate r)
+//   a = exp(rate * r);  S <- a S + sqrt(1 - a^2) i u          1 - a^2 = -e (2 + e), e = expm1(rate r)
 //   out = S * gelu_tanh(y)                                    rounded to the compute dtype for the output product
 // All of it is float32 whatever the compute dtype; the gates' matrices may be bfloat16, and the tensor cores then take
 // the float32 rows u in two bfloat16 parts (u = hi + lo to 16 bits of mantissa), with float32 sums.
@@ -12,9 +12,9 @@
 // in row p % taps, so a step that brings one token writes a row that none of its own readers needs.
 //
 // Three kernels for prompts (conv, gates, scan) and one for decode steps (step).  The scan runs over time in parallel: a
-// block owns 32 channels of a sequence, a warp a stretch of tokens; every warp reduces its stretch to (product of a, end
-// value from zero), the stretches are chained in shared memory, and every warp runs its tokens again from the value it is
-// handed, from registers.  Nothing depends on the other sequences of a step.
+// block owns 16 channels of a sequence, half a warp a stretch of tokens; every stretch is reduced to (product of a, end
+// value from zero), the stretches are chained in shared memory, and every stretch runs its tokens again from the value it
+// is handed, from registers.  Nothing depends on the other sequences of a step.
 #include <math.h>
 
 #include "common.cuh"
@@ -39,12 +39,22 @@ struct Lru {
   int ld, ldo, n_tokens, n_seqs, width, blocks, taps, state_stride, write_state, max_new;
 };
 
-__device__ __forceinline__ float lru_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ __forceinline__ float lru_gelu(float z) { return activate(z, STRATUM_ACT_GELU_TANH); }
-// (a, b) of S <- a S + b
+// FAST: exponential and quotient of the special function unit (a few units in the last place of float32) instead of the
+// library's, on the bfloat16 path.
+template <bool FAST>
+__device__ __forceinline__ float lru_sigmoid(float z) {
+  return FAST ? __fdividef(1.0f, 1.0f + __expf(-z)) : 1.0f / (1.0f + expf(-z));
+}
+template <bool FAST>
+__device__ __forceinline__ float lru_gelu(float z) {   // (1 + tanh w) / 2 = sigmoid(2 w)
+  if (!FAST) return activate(z, STRATUM_ACT_GELU_TANH);
+  return z * lru_sigmoid<true>(1.59576912160573071176f * (z + 0.044715f * z * z * z));
+}
+// (a, b) of S <- a S + b.  Both from e = a - 1, which keeps its digits where a is nearly one: 1 - a^2 = -e (2 + e).
+template <bool FAST>
 __device__ __forceinline__ float2 lru_coefficients(float r_pre, float i_pre, float u, float rate) {
-  const float la = rate * lru_sigmoid(r_pre);
-  return make_float2(expf(la), sqrtf(-expm1f(2.0f * la)) * lru_sigmoid(i_pre) * u);
+  const float e = expm1f(rate * lru_sigmoid<FAST>(r_pre));
+  return make_float2(1.0f + e, sqrtf(-e * (2.0f + e)) * lru_sigmoid<FAST>(i_pre) * u);
 }
 
 // ---------------------------------------------------------------- conv: a thread per (run of tokens, channel)
@@ -217,19 +227,21 @@ __global__ void __launch_bounds__(256) lru_gates_kernel(const Lru P) {
 }
 
 // ---------------------------------------------------------------- scan
-#define LS_TOKENS 8           // tokens of a warp's stretch
+#define LS_TOKENS 8           // tokens of a stretch
+#define LS_CHANNELS 16        // channels of a block: two stretches a warp
 #define LS_MAX_WARPS 16
 
 template <typename T>
-__global__ void __launch_bounds__(LS_MAX_WARPS * 32) lru_scan_kernel(const Lru P) {
-  __shared__ float ends[2][LS_MAX_WARPS][2][32];     // product of a, end value from zero
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
-  const int seq = blockIdx.y, c = blockIdx.x * 32 + lane;
+__global__ void __launch_bounds__(LS_MAX_WARPS * 32, 2) lru_scan_kernel(const Lru P) {
+  constexpr bool FAST = sizeof(T) == 2;
+  __shared__ float2 ends[2][2 * LS_MAX_WARPS][LS_CHANNELS];      // product of a, end value from zero
+  const int stretch = threadIdx.x / LS_CHANNELS, lane = threadIdx.x % LS_CHANNELS, n_stretches = blockDim.x / LS_CHANNELS;
+  const int seq = blockIdx.y, c = blockIdx.x * LS_CHANNELS + lane;
   const int r0 = P.seq_start[seq], r1 = P.seq_start[seq + 1];
   if (r0 >= r1) return;
   const bool live = c < P.width;
   if (P.token_seq[r0] < 0) {                         // rows of no sequence: nothing is kept, the output is zero
-    for (int r = r0 + warp; r < r1; r += n_warps)
+    for (int r = r0 + stretch; r < r1; r += n_stretches)
       if (live) ((T*)P.out)[(size_t)r * P.ldo + c] = from_float<T>(0.f);
     return;
   }
@@ -237,10 +249,10 @@ __global__ void __launch_bounds__(LS_MAX_WARPS * 32) lru_scan_kernel(const Lru P
   const int col_r = (cc / size) * size + cc, col_i = col_r + size;      // 2 size b + (c - size b), then i's
   float* slot = P.state + (size_t)P.seq_slot[seq] * P.state_stride;
   const float rate = P.rate[cc], bias_r = P.gate_b[col_r], bias_i = P.gate_b[col_i];
-  float S = live ? slot[cc] : 0.f;                   // the value in front of the round, the same in every warp
+  float S = live ? slot[cc] : 0.f;                   // the value in front of the round, the same in every stretch
   int buf = 0;
-  for (int base = r0; base < r1; base += n_warps * LS_TOKENS, buf ^= 1) {
-    const int t0 = base + warp * LS_TOKENS;
+  for (int base = r0; base < r1; base += n_stretches * LS_TOKENS, buf ^= 1) {
+    const int t0 = base + stretch * LS_TOKENS;
     float a[LS_TOKENS], b[LS_TOKENS], yv[LS_TOKENS];
     float uu[LS_TOKENS], rr[LS_TOKENS], ii[LS_TOKENS];
 #pragma unroll
@@ -255,28 +267,29 @@ __global__ void __launch_bounds__(LS_MAX_WARPS * 32) lru_scan_kernel(const Lru P
     float A = 1.f, H = 0.f;
 #pragma unroll
     for (int j = 0; j < LS_TOKENS; j++) {
-      const float2 ab = lru_coefficients(rr[j] + bias_r, ii[j] + bias_i, uu[j], rate);
+      const float2 ab = lru_coefficients<FAST>(rr[j] + bias_r, ii[j] + bias_i, uu[j], rate);
       const bool ok = t0 + j < r1;
       a[j] = ok ? ab.x : 1.f;
       b[j] = ok ? ab.y : 0.f;
       A *= a[j];
       H = fmaf(a[j], H, b[j]);
     }
-    ends[buf][warp][0][lane] = A;
-    ends[buf][warp][1][lane] = H;
+    ends[buf][stretch][lane] = make_float2(A, H);
     __syncthreads();                                 // (the other buffer's readers are past their loop: one barrier a round)
     float mine = S;
-    for (int w = 0; w < n_warps; w++) {
-      if (w == warp) mine = S;
-      S = fmaf(ends[buf][w][0][lane], S, ends[buf][w][1][lane]);
+#pragma unroll 8
+    for (int w = 0; w < n_stretches; w++) {
+      if (w == stretch) mine = S;
+      const float2 e = ends[buf][w][lane];
+      S = fmaf(e.x, S, e.y);
     }
 #pragma unroll
     for (int j = 0; j < LS_TOKENS; j++) {
       mine = fmaf(a[j], mine, b[j]);
-      if (live && t0 + j < r1) ((T*)P.out)[(size_t)(t0 + j) * P.ldo + c] = from_float<T>(mine * lru_gelu(yv[j]));
+      if (live && t0 + j < r1) ((T*)P.out)[(size_t)(t0 + j) * P.ldo + c] = from_float<T>(mine * lru_gelu<FAST>(yv[j]));
     }
   }
-  if (P.write_state && live && warp == 0) {
+  if (P.write_state && live && stretch == 0) {
     slot[c] = S;
     const int keep = min(P.taps, r1 - r0);           // the ring takes the step's last inputs
     for (int k = 0; k < keep; k++) {
@@ -407,9 +420,9 @@ __global__ void __launch_bounds__(LT_WARPS * 32) lru_step_kernel(const Lru P) {
       const float rp = acc[n][e] + part[((quad * 2 + n) * 4 + e) * 32 + lane];
       const float ip = acc[n][2 + e] + part[((quad * 2 + n) * 4 + 2 + e) * 32 + lane];
       float* slot = P.state + (size_t)P.seq_slot[seq] * P.state_stride;
-      const float2 ab = lru_coefficients(rp + bias_r, ip + bias_i, u_own[m * LT_CHANNELS + ch - c0], rate);
+      const float2 ab = lru_coefficients<true>(rp + bias_r, ip + bias_i, u_own[m * LT_CHANNELS + ch - c0], rate);
       const float S = fmaf(ab.x, ld_fresh(slot + chan), ab.y);
-      *o = __float2bfloat16_rn(S * lru_gelu(ld_fresh(P.y + (size_t)row * P.ld + chan)));
+      *o = __float2bfloat16_rn(S * lru_gelu<true>(ld_fresh(P.y + (size_t)row * P.ld + chan)));
       if (P.write_state) {
         slot[chan] = S;
         slot[(size_t)(1 + P.token_pos[row] % P.taps) * P.width + chan] = ld_fresh(P.x + (size_t)row * P.ld + chan);
@@ -469,9 +482,9 @@ STRATUM_EXPORT int stratum_lru_scan(const Lru* params, int out_dtype, cudaStream
   if (P.n_tokens <= 0 || P.n_seqs <= 0) return 0;
   const int bad = lru_check(P);
   if (bad) return bad;
-  int warps = (P.max_new + LS_TOKENS - 1) / LS_TOKENS;
+  int warps = (P.max_new + 2 * LS_TOKENS - 1) / (2 * LS_TOKENS);
   warps = warps < 1 ? 1 : (warps > LS_MAX_WARPS ? LS_MAX_WARPS : warps);
-  const dim3 grid((P.width + 31) / 32, P.n_seqs);
+  const dim3 grid((P.width + LS_CHANNELS - 1) / LS_CHANNELS, P.n_seqs);
   if (out_dtype == STRATUM_DT_F32) lru_scan_kernel<float><<<grid, warps * 32, 0, stream>>>(P);
   else if (out_dtype == STRATUM_DT_BF16) lru_scan_kernel<bf16><<<grid, warps * 32, 0, stream>>>(P);
   else return STRATUM_ERR_DTYPE;

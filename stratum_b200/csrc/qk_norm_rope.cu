@@ -13,6 +13,8 @@
 // Everything between the projection's sums and the rounding of the results is float32.  Tokens of no sequence
 // (sequence index -1) write nothing to the caches.  One block per token; the block's shape is fixed, so a row's sums
 // do not depend on the step.
+// Rows in multiples of four values (16-byte aligned) take a form that reads the row once, into shared memory, as vectors,
+// and evaluates every angle of the token once.
 #include <math.h>
 
 #include "common.cuh"
@@ -119,6 +121,103 @@ __global__ void __launch_bounds__(QK_THREADS) qk_norm_rope_kernel(const QKNormRo
   }
 }
 
+// The form for rows in multiples of four values.
+#define QK_ROW_THREADS 512
+__device__ __forceinline__ void qk_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void qk_store4(bf16* p, float4 v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<const uint32_t*>(&a);
+  u.y = *reinterpret_cast<const uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(QK_ROW_THREADS) qk_norm_rope_row_kernel(const QKNormRope P) {
+  extern __shared__ __align__(16) float qk_row[];    // the row's queries and keys | cos, sin | 1 / rms per head
+  __shared__ float sums[2][QK_ROW_THREADS / 32];
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int D = P.dim, nq = P.n_heads * D, nk = P.n_kv * D, nv = P.n_kv * P.v_dim, heads = P.n_heads + P.n_kv;
+  float2* cs = reinterpret_cast<float2*>(qk_row + nq + nk);
+  float* mul = reinterpret_cast<float*>(cs + P.rot_pairs);
+  pdl_trigger();
+  const int pos = P.token_pos[t], seq = P.token_seq[t];
+  for (int i = threadIdx.x; i < P.rot_pairs; i += QK_ROW_THREADS) {
+    float sn, c;
+    sincosf((float)pos * P.inv_freq[i], &sn, &c);
+    cs[i] = make_float2(c, sn);
+  }
+  const int page = P.write_cache && seq >= 0 ? P.block_table[(size_t)seq * P.bt_stride + pos / P.page_tokens] : -1;
+  const int in_page = pos % P.page_tokens;
+  const float* row = P.proj + (size_t)t * P.ld;
+  pdl_wait();                                        // the projection is the work of the kernel before: ld_fresh
+  float ssq = 0.f, ssk = 0.f;
+  for (int c = 4 * threadIdx.x; c < nq + nk; c += 4 * QK_ROW_THREADS) {
+    const float4 v = ld_fresh(reinterpret_cast<const float4*>(row + c));
+    *reinterpret_cast<float4*>(qk_row + c) = v;
+    const float s = fmaf(v.w, v.w, fmaf(v.z, v.z, fmaf(v.y, v.y, v.x * v.x)));
+    if (c < nq) ssq += s; else ssk += s;
+  }
+  if (page >= 0) {                                   // values: no norm, no rotation
+    for (int c = 4 * threadIdx.x; c < nv; c += 4 * QK_ROW_THREADS) {
+      const int h = c / P.v_dim, d = c - h * P.v_dim;
+      qk_store4((T*)P.v_cache + (((size_t)page * P.n_kv + h) * P.page_tokens + in_page) * P.v_dim + d,
+                ld_fresh(reinterpret_cast<const float4*>(row + nq + nk + c)));
+    }
+  }
+  if (P.per_head) {
+    __syncthreads();
+    for (int h = warp; h < heads; h += QK_ROW_THREADS / 32) {          // a head's sum: one warp, one order
+      float ss = 0.f;
+      for (int d = lane; d < D; d += 32) ss = fmaf(qk_row[h * D + d], qk_row[h * D + d], ss);
+      ss = warp_sum(ss);
+      if (lane == 0) mul[h] = 1.0f / sqrtf(ss / (float)D + P.eps);
+    }
+    __syncthreads();
+  } else {
+    ssq = warp_sum(ssq);
+    ssk = warp_sum(ssk);
+    if (lane == 0) { sums[0][warp] = ssq; sums[1][warp] = ssk; }
+    __syncthreads();
+    ssq = ssk = 0.f;
+#pragma unroll
+    for (int w = 0; w < QK_ROW_THREADS / 32; w++) { ssq += sums[0][w]; ssk += sums[1][w]; }
+    ssq = 1.0f / sqrtf(ssq / (float)nq + P.eps);
+    ssk = 1.0f / sqrtf(ssk / (float)nk + P.eps);
+  }
+  T* qo = (T*)P.q_out + (size_t)t * P.ldq;
+  const int rp = P.rot_pairs, last = page >= 0 ? nq + nk : nq;
+  for (int c = 4 * threadIdx.x; c < last; c += 4 * QK_ROW_THREADS) {
+    const bool is_q = c < nq;
+    const int h = c / D, d0 = c - h * D;             // heads of queries, then of keys
+    const float m = P.per_head ? mul[h] : (is_q ? ssq : ssk);
+    const float* gain = is_q ? P.q_gain : P.k_gain;
+    const int g0 = P.per_head ? d0 : (is_q ? c : c - nq);
+    float out[4];
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      const int d = d0 + i;
+      float v = qk_row[c + i] * m * gain[g0 + i];
+      if (d < 2 * rp) {
+        const bool second = P.half ? d >= rp : d & 1;
+        const int step = P.half ? (second ? -rp : rp) : (second ? -1 : 1), pair = P.half ? (second ? d - rp : d) : d >> 1;
+        const float w = qk_row[c + i + step] * m * gain[g0 + i + step];
+        const float2 f = cs[pair];
+        v = (second ? v * f.x + w * f.y : v * f.x - w * f.y) * P.magnitude;
+      }
+      out[i] = v;
+    }
+    const float4 v4 = make_float4(out[0], out[1], out[2], out[3]);
+    if (is_q) {
+      qk_store4(qo + c, v4);
+    } else {
+      const size_t at = (((size_t)page * P.n_kv + h - P.n_heads) * P.page_tokens + in_page) * D + d0;
+      qk_store4((T*)P.k_cache + at, v4);
+      if (P.v_dim == 0) qk_store4((T*)P.v_cache + at, *reinterpret_cast<const float4*>(qk_row + c));
+    }
+  }
+}
+
 STRATUM_EXPORT int stratum_qk_norm_rope(const QKNormRope* params, int dtype, cudaStream_t stream) {
   const QKNormRope& P = *params;
   if (P.n_tokens <= 0) return 0;
@@ -128,6 +227,19 @@ STRATUM_EXPORT int stratum_qk_norm_rope(const QKNormRope* params, int dtype, cud
     return STRATUM_ERR_SHAPE;
   const size_t smem = P.per_head ? (size_t)(P.n_heads + P.n_kv) * sizeof(float) : 0;
   if (smem > 40 * 1024) return STRATUM_ERR_LIMIT;
+  // (which form: by sizes and alignment alone, which a model's buffers share from step to step)
+  const uintptr_t bits = (uintptr_t)P.proj | (uintptr_t)P.q_out | (uintptr_t)P.k_cache | (uintptr_t)P.v_cache;
+  const size_t row_smem = ((size_t)(P.n_heads + P.n_kv) * (P.dim + 1) + 2 * (size_t)P.rot_pairs) * sizeof(float);
+  if (P.dim % 4 == 0 && P.v_dim % 4 == 0 && P.ld % 4 == 0 && P.ldq % 4 == 0 && (bits & 15) == 0 && row_smem <= 100 * 1024 &&
+      (dtype == STRATUM_DT_F32 || dtype == STRATUM_DT_BF16)) {
+    void (*kern)(const QKNormRope) = dtype == STRATUM_DT_F32 ? qk_norm_rope_row_kernel<float> : qk_norm_rope_row_kernel<bf16>;
+    if (row_smem > 40 * 1024) {
+      cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)row_smem);
+      if (e != cudaSuccess) return (int)e;
+    }
+    launch_pdl(kern, P.n_tokens, QK_ROW_THREADS, row_smem, stream, P);
+    return launch_status();
+  }
   if (dtype == STRATUM_DT_F32) launch_pdl(qk_norm_rope_kernel<float>, P.n_tokens, QK_THREADS, smem, stream, P);
   else if (dtype == STRATUM_DT_BF16) launch_pdl(qk_norm_rope_kernel<bf16>, P.n_tokens, QK_THREADS, smem, stream, P);
   else return STRATUM_ERR_DTYPE;

@@ -1093,7 +1093,8 @@ class GlaStep:
     [tokens, heads * vdim]; `finish(...)` norms and gates them into out (compute dtype [tokens, >= heads * vdim]).
 
     With head_decay (float32 [heads]: a constant decay per head; rank 0) there is neither `cast` nor `decay`;
-    `rotate(table, interleaved)` turns q and k in place by the step's (cos, sin) table float32 [tokens, pairs, 2]."""
+    `rotate(table, interleaved)` turns q and k in place by the step's (cos, sin) table float32 [tokens, pairs, 2], and
+    `recur` may take the tokens in chunks on tensor cores (`chunked`; see csrc/gla_chunked.cu) where `chunks_ok`."""
 
     def __init__(self, proj: torch.Tensor, n_heads: int, dim: int, vdim: int, rank: int, tau: float, q_scale: float,
                  eps: float, head_decay: Optional[torch.Tensor] = None):
@@ -1112,6 +1113,11 @@ class GlaStep:
                 raise KernelError("gla: one decay per head")
             p.head_decay = head_decay.data_ptr()
             self.keep.append(head_decay)
+
+    def chunks_ok(self) -> bool:
+        p = self.p
+        return bool(p.head_decay) and p.dim % 16 == 0 and p.dim <= 256 and p.vdim % 4 == 0 and p.ld % 4 == 0 \
+            and p.proj % 16 == 0
 
     def rotate(self, table: torch.Tensor, interleaved: bool) -> None:
         _need(table, "table", torch.float32)
@@ -1142,7 +1148,7 @@ class GlaStep:
         self._run(0, torch.float32, "gla_decay")
 
     def recur(self, o_raw: torch.Tensor, state: torch.Tensor, token_seq: torch.Tensor, seq_start: torch.Tensor,
-              seq_slot: torch.Tensor, write_state: bool = True) -> None:
+              seq_slot: torch.Tensor, write_state: bool = True, chunked: bool = False) -> None:
         _need(o_raw, "o_raw", torch.float32); _need(state, "state", torch.float32)
         _need(token_seq, "token_seq", torch.int32); _need(seq_start, "seq_start", torch.int32)
         _need(seq_slot, "seq_slot", torch.int32)
@@ -1152,6 +1158,10 @@ class GlaStep:
         p.o_raw, p.state, p.state_stride = o_raw.data_ptr(), state.data_ptr(), state.stride(0)
         p.token_seq, p.seq_start, p.seq_slot = token_seq.data_ptr(), seq_start.data_ptr(), seq_slot.data_ptr()
         p.n_seqs, p.write_state = seq_slot.numel(), int(bool(write_state))
+        if chunked:
+            f = _fn("gla_chunked", "stratum_gla_chunked", [c_void_p, c_void_p])
+            _check(f(ctypes.addressof(p), _stream()), "gla_chunked")
+            return
         self._run(1, torch.float32, "gla_recur")
 
     def finish(self, gain: Optional[torch.Tensor], out: torch.Tensor) -> None:
@@ -1457,22 +1467,30 @@ def attention_tile(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
 
 def attention_tc(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, token_pos: torch.Tensor,
                  block_table: torch.Tensor, qblocks, out: torch.Tensor, n_q: int, n_kv: int, head_dim: int,
-                 page_tokens: int, window: int, scale: float, halves: int = 1) -> None:
+                 page_tokens: int, window: int, scale: float, halves: int = 1, split: bool = False, chunk: int = 0,
+                 gate: Optional[torch.Tensor] = None) -> None:
     """bfloat16 attention for prompts on tcgen05/TMEM: query tiles of halves * 128 / (n_q / n_kv) tokens (qblocks
     as for attention_tile).  halves 2: a CTA owns 256 query rows whose two halves share every key and value tile.
-    head_dim 64 or 128, group size dividing 128, pages of 64 tokens."""
+    head_dim 64 or 128, group size dividing 128, pages of 64 tokens.  split (with halves 2): the probabilities keep 16
+    bits of mantissa (two bfloat16 parts) instead of 8; chunk: a position sees only keys of its own chunk of that many
+    positions (0: all); gate (float32 [tokens, n_q * head_dim]): the output times sigmoid(gate), element by element."""
+    if gate is not None:
+        _need(gate, "gate", torch.float32, contiguous=False)
+        if gate.shape[0] != qkv.shape[0] or gate.shape[1] < n_q * head_dim or gate.stride(1) != 1:
+            raise KernelError("attention_tc: the output gate has a column per head and value dimension")
     _need(qkv, "qkv", torch.bfloat16); _need(k_cache, "k_cache", torch.bfloat16)
     _need(v_cache, "v_cache", torch.bfloat16); _need(out, "out", torch.bfloat16)
     _need(block_table, "block_table", torch.int32)
     qs, qt, qn = qblocks
     f = _fn("attention_tc", "stratum_attention_tc",
             [c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-             c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
-             c_void_p])
+             c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int,
+             c_void_p, c_int, c_void_p, c_void_p])
     _check(f(_ptr(qkv), qkv.stride(0), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0], _ptr(token_pos),
              _ptr(block_table), block_table.stride(0), _ptr(qs), _ptr(qt), _ptr(qn), qs.numel(), _ptr(out),
              out.stride(0), qkv.shape[0], n_q, n_kv, head_dim, page_tokens, window, c_float(scale), halves,
-             _ptr(status_word()), _stream()), "attention_tc")
+             int(bool(split)), int(chunk), _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(status_word()),
+             _stream()), "attention_tc")
 
 
 _stream_scratch = None

@@ -115,13 +115,31 @@ def run_general_dense(att, shape, q: torch.Tensor, keys: torch.Tensor, values: t
                             seq_start=step.seq_start)
 
 
+def _plain_heads(shape, q: torch.Tensor, cache, out: torch.Tensor, gate) -> bool:
+    """Whether a general attention is one the tcgen05 prompt kernel knows: keys and values of one size, 64 or 128, one map
+    per head, groups that divide 128, no sink, kept first keys, cap or factor on the scores beside a positive scale."""
+    return (q.dtype == torch.bfloat16 and shape.maps == 1 and not shape.v_in_k and shape.qk_dim == shape.v_dim
+            and shape.qk_dim in (64, 128) and 128 % shape.group == 0 and shape.sink is None and shape.head_scale is None
+            and not shape.keep_first and not shape.softcap and not shape.temp_coef and shape.scale > 0
+            and q.is_contiguous() and out.is_contiguous() and q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0
+            and (gate is None or (gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0)))
+
+
 def run_general(att, shape, q: torch.Tensor, cache, step, out: torch.Tensor, gate=None) -> None:
     """Attention of the shapes kernels.AttentionShape describes (key and value sizes of their own, values inside the
     key rows, several maps per head): q [tokens, *] holds head j's map m at column (j * maps + m) * qk_dim.
-    bfloat16 with sizes in multiples of 8: the tensor-core kernel (decode steps: the keys cut into ranges that
+    bfloat16 prompts of heads that need nothing beyond chunks, a window and a gate: the tcgen05 kernel, with
+    probabilities of 16 bits; bfloat16 with sizes in multiples of 8: the tensor-core kernel (decode steps: the keys cut into ranges that
     fill the GPU; prompts: query blocks of 16 rows); everything else: the CUDA-core kernel, float32 throughout.
     gate (float32 [tokens, heads * v_dim] or None): pre-activations of an output gate per element.
-    STRATUM_GENERAL_ATTENTION_MMA=0: always the CUDA-core kernel (measurements)."""
+    STRATUM_GENERAL_ATTENTION_TC=0: not the tcgen05 kernel; STRATUM_GENERAL_ATTENTION_MMA=0: always the CUDA-core kernel
+    (measurements)."""
+    if not step.all_single and _plain_heads(shape, q, cache, out, gate) \
+            and os.environ.get("STRATUM_GENERAL_ATTENTION_TC", "1") != "0":
+        K.attention_tc(q, cache.k, cache.v, step.token_pos, cache.block_table, step.query_blocks(2 * (128 // shape.group)),
+                       out, shape.n_heads, shape.n_heads // shape.group, shape.qk_dim, PAGE_TOKENS, shape.window, shape.scale,
+                       halves=2, split=True, chunk=shape.chunk, gate=gate)
+        return
     if (not K.attention_general_mma_ok(shape, q, out, PAGE_TOKENS, gate)
             or os.environ.get("STRATUM_GENERAL_ATTENTION_MMA", "1") == "0"):
         K.attention_general(shape, q, cache.k, cache.v, step.token_pos, step.token_seq, cache.block_table, out,

@@ -10,7 +10,8 @@ Head j, with its constant decay c_j:
     o <- o / sqrt(mean(o^2) + eps) * silu(Wg h)_j;     result = Wo concat_j(o)
 
 The four projections run as one product with float32 sums; everything from there to the output product is float32
-(csrc/gla.cu, the kernels of gated linear attention with a decay per head in place of one per token and key channel).
+(csrc/gla.cu, the kernels of gated linear attention with a decay per head in place of one per token and key channel; the
+prompts of the bfloat16 path go chunk by chunk through tensor cores, csrc/gla_chunked.cu).
 """
 from __future__ import annotations
 
@@ -25,6 +26,9 @@ from .latent_attention import padded
 from .linear import ADD_TO_F32, STORE_F32, Linear
 from .registry import find_part, register_part
 from .spec import PartSpec, TensorSpec
+
+
+CHUNKED_FROM = 16             # new tokens of a sequence from which a step goes through chunks
 
 
 @register_part("mixer", "retention")
@@ -79,7 +83,8 @@ class Retention(Mixer):
             rot = self.position.rotary()
             step_.rotate(step.rotation_table(rot), rot.interleaved)
         o_raw = self.runtime.empty(T, self.v_cols, dtype=f32)
-        step_.recur(o_raw, cache.state, step.token_seq, step.seq_start, step.seq_slot, cache.writes)
+        chunked = xin.dtype == torch.bfloat16 and step.max_new >= CHUNKED_FROM and step_.chunks_ok()
+        step_.recur(o_raw, cache.state, step.token_seq, step.seq_start, step.seq_slot, cache.writes, chunked)
         out = self.runtime.empty(T, padded(self.v_cols))
         step_.finish(None, out)
         self.w_o(out[:, :self.v_cols], out=residual, mode=STORE_F32 if store else ADD_TO_F32)

@@ -118,6 +118,11 @@ class SinkAttention(Mixer):
             self.w_in = Linear(self.runtime, *self.input_weights(weights))
         self.w_o = Linear(self.runtime, weights[n["o"]])
         self.q_gain, self.k_gain = weights[n["q_norm"]].contiguous(), weights[n["k_norm"]].contiguous()
+        # a factor per head on the scores rides on the queries' gain where that has a value per column
+        temp = weights[n["temp"]].contiguous() if self.has_temp else None
+        if temp is not None and not self.per_head:
+            self.q_gain = (self.q_gain.view(self.n_heads, self.d) * temp[:, None]).reshape(-1).contiguous()
+            temp = None
         self.sink = None
         if self.has_sink:
             self.sink = weights[n["sink"]].contiguous()
@@ -125,7 +130,7 @@ class SinkAttention(Mixer):
             self.sink = torch.zeros(self.n_heads, dtype=torch.float32, device=self.q_gain.device)
         self.shape = K.AttentionShape(self.n_heads, self.n_heads // self.n_kv, 1, self.d, self.dv, False, self.scale,
                                       window=self.window, sink=self.sink, keep_first=self.keep_first, chunk=self.chunk,
-                                      head_scale=weights[n["temp"]].contiguous() if self.has_temp else None)
+                                      head_scale=temp)
 
     def cache_spec(self) -> KVSpec:
         order = "normed_rotated" + ("_half" if self.half else "") + ("" if self.own_values else "_values_raw")

@@ -121,13 +121,18 @@ def test_clamped_gate_rides_on_every_product(M, N, K_):
 
 
 @pytest.mark.parametrize("heads,dim,vdim,pairs", [(3, 12, 20, 4), (2, 40, 8, 20), (1, 9, 7, 0), (4, 64, 32, 32), (2, 130, 70, 10),
-                                                  (1, 260, 8, 2), (2, 128, 128, 64), (8, 64, 64, 16)])
+                                                  (1, 260, 8, 2), (2, 128, 128, 64), (8, 64, 64, 16), (2, 256, 36, 128),
+                                                  (1, 208, 100, 0), (3, 16, 4, 8)])
 @pytest.mark.parametrize("long", [77, 520])
-@pytest.mark.parametrize("interleaved", [False, True])
-def test_retention_kernels(heads, dim, vdim, pairs, long, interleaved):
+@pytest.mark.parametrize("form", ["tokens", "tokens, neighbouring pairs", "chunks"])
+def test_retention_kernels(heads, dim, vdim, pairs, long, form):
     """Rotation, recurrence with a constant decay per head and the heads' norm on projections made here: two sequences of
-    unequal lengths whose tokens come in four steps (many, one of each, three and two, one), in slots that lie apart."""
+    unequal lengths whose tokens come in four steps (many, one of each, three and two, one), in slots that lie apart; the
+    recurrence token by token, and in chunks on tensor cores where sizes allow."""
     from stratum_b200 import kernels as K
+    interleaved = form.endswith("pairs")
+    if form == "chunks" and (dim % 16 or dim > 256):
+        pytest.skip("sizes the chunked form does not take")
     rng = np.random.default_rng(dim + vdim)
     HD, HV = heads * dim, heads * vdim
     lens = (long, 11)
@@ -144,7 +149,7 @@ def test_retention_kernels(heads, dim, vdim, pairs, long, interleaved):
         want = [G.retention(m, 1e-5, w, p[:, cols], "") for p in proj]
     else:
         want = [G.retention(m, 1e-5, w, p, "") for p in proj]
-    st = torch.zeros(6, HD * vdim + 3, device="cuda")
+    st = torch.zeros(6, HD * vdim + 4, device="cuda")
     slots, done, got = (4, 1), [0, 0], [[], []]
     for cut in ((long - 5, 7), (1, 1), (3, 2), (1, 1)):
         rows = np.concatenate([proj[i][done[i]:done[i] + cut[i]] for i in range(2)])
@@ -157,7 +162,9 @@ def test_retention_kernels(heads, dim, vdim, pairs, long, interleaved):
             g.rotate(_dev(np.stack([np.cos(ang), np.sin(ang)], axis=-1)), interleaved)
         o_raw = torch.empty(T, HV, device="cuda")
         out = torch.empty(T, HV + 5, device="cuda")
-        g.recur(o_raw, st, _i32(seq), _i32([0, cut[0], T]), _i32(slots), True)
+        if form == "chunks":
+            assert g.chunks_ok()
+        g.recur(o_raw, st, _i32(seq), _i32([0, cut[0], T]), _i32(slots), True, chunked=form == "chunks")
         g.finish(None, out)
         o = out[:, :HV].cpu().numpy()
         got[0].append(o[:cut[0]]); got[1].append(o[cut[0]:])
@@ -244,8 +251,19 @@ def test_linear_recurrence_kernels(width, blocks, taps, dtype):
     assert torch.equal(before, state)
 
 
+def _softmax(q, k, v, vis, scales):
+    T, H, _ = q.shape
+    out = np.zeros((T, H, v.shape[2]))
+    for h in range(H):
+        g = h // (H // k.shape[1])
+        s = np.where(vis, q[:, h] @ k[:, g].T * scales[h], -np.inf)
+        e = np.exp(s - s.max(-1, keepdims=True))
+        out[:, h] = e / e.sum(-1, keepdims=True) @ v[:, g]
+    return out.reshape(T, -1)
+
+
 @pytest.mark.parametrize("H,Gk,D,Dv,chunk", [(4, 2, 12, 20, 50), (3, 3, 20, 22, 5), (8, 1, 64, 64, 130), (4, 4, 32, 48, 64),
-                                             (4, 2, 128, 128, 100), (2, 1, 64, 64, 1), (20, 1, 32, 32, 77)])
+                                             (4, 2, 128, 128, 100), (2, 1, 64, 64, 1), (20, 1, 32, 32, 77), (8, 2, 64, 64, 200), (2, 2, 128, 128, 64)])
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_chunked_attention_with_head_factors_and_an_output_gate(H, Gk, D, Dv, chunk, dtype):
     """A paged cache whose pages lie in no order, queries at every position in blocks (prompt) and single queries at
@@ -260,17 +278,15 @@ def test_chunked_attention_with_head_factors_and_an_output_gate(H, Gk, D, Dv, ch
     gate, temp, scale = rng.standard_normal((T, H * Dv)) * 2, rng.uniform(0.3, 2.5, H), 1.5 / np.sqrt(D)
     temp[0] = -0.7
     vis = G.visible(T, chunk)
-    want = np.zeros((T, H, Dv))
-    for h in range(H):
-        s = np.where(vis, q[:, h] @ k[:, h // (H // Gk)].T * scale * temp[h], -np.inf)
-        e = np.exp(s - s.max(-1, keepdims=True))
-        want[:, h] = e / e.sum(-1, keepdims=True) @ v[:, h // (H // Gk)]
-    want = want.reshape(T, H * Dv) * G.sigmoid(gate)
+    want = _softmax(q, k, v, vis, scale * temp) * G.sigmoid(gate)
     pages = [7, 2, 9, 4, 0, 5]
     kc, vc = np.zeros((10, Gk, 64, D)), np.zeros((10, Gk, 64, Dv))
     for t in range(T):
         kc[pages[t // 64], :, t % 64], vc[pages[t // 64], :, t % 64] = k[t], v[t]
     kc, vc = _dev(kc, td), _dev(vc, td)
+    if D == Dv and D in (64, 128):
+        temp[:] = 1.0                                        # (the tcgen05 kernel takes no factor per head)
+        want = _softmax(q, k, v, vis, np.full(H, scale)) * G.sigmoid(gate)
     shape = K.AttentionShape(H, H // Gk, 1, D, Dv, False, scale, chunk=chunk, head_scale=_dev(temp))
     bt = _i32([pages])
     tol = 2e-5 if dtype == "float32" else 1e-2
@@ -307,6 +323,16 @@ def test_chunked_attention_with_head_factors_and_an_output_gate(H, Gk, D, Dv, ch
                     K.attention_general_mma(shape, qd, kc, vc, pos, seq, tables, out, 64, qb, per_block, 1, 384, None, None,
                                             groups, gate=gd)
                     yield out[:, :H * Dv].double().cpu().numpy()
+        if D == Dv and D in (64, 128) and td == torch.bfloat16 and not single:      # the tcgen05 kernel
+            b = 2 * (128 // (H // Gk))
+            starts = np.arange(0, n, b)
+            qb = (torch.zeros(len(starts), dtype=torch.int32, device="cuda"), _i32(starts), _i32(np.minimum(b, n - starts)))
+            out.zero_()
+            K.attention_tc(qd, kc, vc, pos, bt, qb, out, H, Gk, D, 64, 0, scale, halves=2, split=True, chunk=chunk, gate=gd)
+            K.check_status()
+            got = out[:, :H * Dv].double().cpu().numpy()
+            assert np.max(np.abs(got - want)) <= 5e-3 * np.max(np.abs(want))        # (the output's rounding alone)
+            yield got
         out.zero_()
         K.attention_general(shape, qd, kc, vc, pos, seq, tables, out, 64, gd)
         yield out[:, :H * Dv].double().cpu().numpy()
