@@ -9,7 +9,7 @@
 // sums, so a product is as good as its factors' 16 bits; the scores q . k and their decays are float32 between the two
 // products they take part in.
 //
-// A CTA of eight warps owns (sequence, head, 32 columns of S).  The next chunk's q, k and v are copied to a staging buffer
+// A CTA owns (sequence, head, 32 columns of S).  The next chunk's q, k and v are copied to a staging buffer
 // (cp.async) while one is worked on; a chunk's phases, each a barrier apart: split into parts; scores; outputs from
 // scores and state; state.  Nothing depends on the other sequences of a step, and on how a sequence's tokens are cut into
 // steps only in the rounding of its sums.
@@ -19,7 +19,6 @@
 #include "gla.h"
 #include "mma_common.cuh"
 
-#define GC_WARPS 8
 #define GC_COLS 32            // columns of S (of v) per CTA
 #define GC_VP 40              // bfloat16 per row of v and S in shared memory: 32 + 8 of padding
 
@@ -67,14 +66,16 @@ __host__ __device__ __forceinline__ size_t gc_smem_bytes(int C, int dim) {
   return floats * 4 + halves * 2;
 }
 
-// C: tokens of a chunk (64 or 32).  MB: blocks of 16 rows of S a warp holds (dim <= 128 MB).
-template <int C, int MB>
-__global__ void __launch_bounds__(GC_WARPS * 32) gla_chunked_kernel(const Gla P) {
+// C: tokens of a chunk (64 or 32).  MB: blocks of 16 rows of S a warp holds (dim <= 128 MB): eight warps cover the rows, and
+// with sixteen the other eight take the other half of the columns.
+template <int C, int MB, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
   extern __shared__ __align__(16) float gc_smem[];
   constexpr int RB = C / 16;                          // blocks of 16 tokens
-  constexpr int CW = GC_WARPS / RB;                   // warps that share a block of tokens
+  constexpr int CW = WARPS / RB;                   // warps that share a block of tokens
   constexpr int NA = C / 8 / CW;                      // blocks of 8 scores a warp takes
   constexpr int NO = GC_COLS / 8 / CW;                // blocks of 8 columns of the output a warp takes
+  constexpr int NS = GC_COLS / 8 / (WARPS / 8);       // blocks of 8 columns of the state a warp holds
   constexpr int AP = C + 8;                           // bfloat16 per row of the scores
   const int D = P.dim, V = P.vdim, HD = P.n_heads * D, HV = P.n_heads * V, QP = D + 8;
   float* stage_q = gc_smem;                           // [C][D]
@@ -107,26 +108,27 @@ __global__ void __launch_bounds__(GC_WARPS * 32) gla_chunked_kernel(const Gla P)
   }
   const float decay = P.head_decay[h];
   for (int m = threadIdx.x; m <= C; m += blockDim.x) power[m] = powf(decay, (float)m);
-  // rows of S that this warp holds: blocks of 16 from 16 (warp + 8 b) on
+  // what this warp holds of S: blocks of 16 rows from 16 (srow + 8 b) on, NS blocks of 8 columns from scol on
+  const int srow = warp % 8, scol = 8 * NS * (warp / 8);
   float* Sg = P.state + (size_t)P.seq_slot[seq] * P.state_stride + ((size_t)h * V + j0) * D;
-  float S[MB][GC_COLS / 8][4];
+  float S[MB][NS][4];
 #pragma unroll
   for (int b = 0; b < MB; b++)
 #pragma unroll
-    for (int n = 0; n < GC_COLS / 8; n++)
+    for (int n = 0; n < NS; n++)
 #pragma unroll
       for (int e = 0; e < 4; e++) {
-        const int d = 16 * (warp + GC_WARPS * b) + g + 8 * (e >> 1), j = 8 * n + 2 * t + (e & 1);
+        const int d = 16 * (srow + 8 * b) + g + 8 * (e >> 1), j = scol + 8 * n + 2 * t + (e & 1);
         S[b][n][e] = (d < D && j0 + j < V) ? Sg[(size_t)j * D + d] : 0.f;
       }
   auto put_state = [&]() {                            // S in two parts, for the products of the next chunk
 #pragma unroll
     for (int b = 0; b < MB; b++) {
-      const int d = 16 * (warp + GC_WARPS * b) + g;
-      if (16 * (warp + GC_WARPS * b) >= D) continue;
+      const int d = 16 * (srow + 8 * b) + g;
+      if (16 * (srow + 8 * b) >= D) continue;
 #pragma unroll
-      for (int n = 0; n < GC_COLS / 8; n++) {
-        const int at = d * GC_VP + 8 * n + 2 * t;
+      for (int n = 0; n < NS; n++) {
+        const int at = d * GC_VP + scol + 8 * n + 2 * t;
         gc_split2(S[b][n][0], S[b][n][1], s_hi + at, s_lo + at);
         gc_split2(S[b][n][2], S[b][n][3], s_hi + at + 8 * GC_VP, s_lo + at + 8 * GC_VP);
       }
@@ -134,9 +136,9 @@ __global__ void __launch_bounds__(GC_WARPS * 32) gla_chunked_kernel(const Gla P)
   };
   put_state();
   auto stage = [&](int c0) {                          // ask for the tokens c0 .. of this sequence; rows beyond it are zero
-    const int n = min(C, r1 - c0), q4 = D / 4;
-    for (int i = threadIdx.x; i < C * q4; i += blockDim.x) {
-      const int tok = i / q4, d = 4 * (i - tok * q4);
+    const int n = min(C, r1 - c0);
+    for (int tok = warp; tok < C; tok += WARPS)
+     for (int d = 4 * lane; d < D; d += 128) {
       float *dq = stage_q + tok * D + d, *dk = stage_k + tok * D + d;
       if (tok < n) {
         const float* row = P.proj + (size_t)(c0 + tok) * P.ld + (size_t)h * D + d;
@@ -161,9 +163,8 @@ __global__ void __launch_bounds__(GC_WARPS * 32) gla_chunked_kernel(const Gla P)
     asm volatile("cp.async.wait_all;" ::: "memory");
     __syncthreads();                                  // the chunk has landed; the parts of the one before are free
     {
-      const int q4 = D / 4;
-      for (int i = threadIdx.x; i < C * q4; i += blockDim.x) {
-        const int tok = i / q4, d = 4 * (i - tok * q4);
+      for (int tok = warp; tok < C; tok += WARPS)
+       for (int d = 4 * lane; d < D; d += 128) {
         gc_split4(*reinterpret_cast<const float4*>(stage_q + tok * D + d), q_hi + tok * QP + d, q_lo + tok * QP + d);
         gc_split4(*reinterpret_cast<const float4*>(stage_k + tok * D + d), k_hi + tok * QP + d, k_lo + tok * QP + d);
       }
@@ -270,10 +271,10 @@ __global__ void __launch_bounds__(GC_WARPS * 32) gla_chunked_kernel(const Gla P)
       const float pn = power[n_here];
 #pragma unroll
       for (int b = 0; b < MB; b++) {
-        const int d0 = 16 * (warp + GC_WARPS * b);
+        const int d0 = 16 * (srow + 8 * b);
         if (d0 >= D) continue;
 #pragma unroll
-        for (int n = 0; n < GC_COLS / 8; n++) { S[b][n][0] *= pn; S[b][n][1] *= pn; S[b][n][2] *= pn; S[b][n][3] *= pn; }
+        for (int n = 0; n < NS; n++) { S[b][n][0] *= pn; S[b][n][1] *= pn; S[b][n][2] *= pn; S[b][n][3] *= pn; }
 #pragma unroll
         for (int kb = 0; kb < RB; kb++) {
           uint32_t ah[4], al[4];
@@ -281,9 +282,9 @@ __global__ void __launch_bounds__(GC_WARPS * 32) gla_chunked_kernel(const Gla P)
           gc_ldsm4_t(ah, k_hi + at);
           gc_ldsm4_t(al, k_lo + at);
 #pragma unroll
-          for (int n = 0; n < GC_COLS / 8; n++) {
+          for (int n = 0; n < NS; n++) {
             uint32_t bh[2], bl[2];
-            const int bt = (16 * kb + (lane & 15)) * GC_VP + 8 * n;
+            const int bt = (16 * kb + (lane & 15)) * GC_VP + scol + 8 * n;
             gc_ldsm2_t(bh, w_hi + bt);
             gc_ldsm2_t(bl, w_lo + bt);
             gc_mma3(S[b][n], ah, al, bh, bl);
@@ -298,23 +299,23 @@ __global__ void __launch_bounds__(GC_WARPS * 32) gla_chunked_kernel(const Gla P)
 #pragma unroll
     for (int b = 0; b < MB; b++)
 #pragma unroll
-      for (int n = 0; n < GC_COLS / 8; n++)
+      for (int n = 0; n < NS; n++)
 #pragma unroll
         for (int e = 0; e < 4; e++) {
-          const int d = 16 * (warp + GC_WARPS * b) + g + 8 * (e >> 1), j = 8 * n + 2 * t + (e & 1);
+          const int d = 16 * (srow + 8 * b) + g + 8 * (e >> 1), j = scol + 8 * n + 2 * t + (e & 1);
           if (d < D && j0 + j < V) Sg[(size_t)j * D + d] = S[b][n][e];
         }
   }
 }
 
-template <int C, int MB>
+template <int C, int MB, int WARPS>
 static int gla_chunked_launch(const Gla& P, cudaStream_t stream) {
   const size_t smem = gc_smem_bytes(C, P.dim);
   if (smem > 225 * 1024) return STRATUM_ERR_LIMIT;
-  cudaError_t e = cudaFuncSetAttribute(gla_chunked_kernel<C, MB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  cudaError_t e = cudaFuncSetAttribute(gla_chunked_kernel<C, MB, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const dim3 grid((P.vdim + GC_COLS - 1) / GC_COLS, P.n_heads, P.n_seqs);
-  gla_chunked_kernel<C, MB><<<grid, GC_WARPS * 32, smem, stream>>>(P);
+  gla_chunked_kernel<C, MB, WARPS><<<grid, WARPS * 32, smem, stream>>>(P);
   return launch_status();
 }
 
@@ -327,7 +328,7 @@ STRATUM_EXPORT int stratum_gla_chunked(const Gla* params, cudaStream_t stream) {
   if (bad) return bad;
   if (!P.head_decay || P.dim % 16 != 0 || P.vdim % 4 != 0 || P.ld % 4 != 0) return STRATUM_ERR_SHAPE;
   if (((uintptr_t)P.proj & 15) != 0 || ((uintptr_t)P.o_raw & 7) != 0) return STRATUM_ERR_ALIGN;
-  if (P.dim <= 128) return gla_chunked_launch<64, 1>(P, stream);
-  if (P.dim <= 256) return gla_chunked_launch<32, 2>(P, stream);
+  if (P.dim <= 128) return gla_chunked_launch<64, 1, 16>(P, stream);
+  if (P.dim <= 256) return gla_chunked_launch<32, 2, 8>(P, stream);
   return STRATUM_ERR_LIMIT;
 }

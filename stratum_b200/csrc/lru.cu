@@ -41,9 +41,30 @@ struct Lru {
 
 // FAST: exponential and quotient of the special function unit (a few units in the last place of float32) instead of the
 // library's, on the bfloat16 path.
+__device__ __forceinline__ float lru_quick_reciprocal(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float lru_quick_root(float x) {
+  float y;
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 template <bool FAST>
 __device__ __forceinline__ float lru_sigmoid(float z) {
-  return FAST ? __fdividef(1.0f, 1.0f + __expf(-z)) : 1.0f / (1.0f + expf(-z));
+  return FAST ? lru_quick_reciprocal(1.0f + __expf(-z)) : 1.0f / (1.0f + expf(-z));
+}
+// exp(x) - 1 for x <= 0: its Taylor series to x^7 where |x| < 1/4 (what is left out is below 2^-29 of the first
+// term), the exponential itself below that, where the difference costs at most three bits
+__device__ __forceinline__ float lru_quick_expm1(float x) {
+  float s = fmaf(x, 1.0f / 5040.0f, 1.0f / 720.0f);
+  s = fmaf(s, x, 1.0f / 120.0f);
+  s = fmaf(s, x, 1.0f / 24.0f);
+  s = fmaf(s, x, 1.0f / 6.0f);
+  s = fmaf(s, x, 0.5f);
+  s = fmaf(s * x, x, x);
+  return x > -0.25f ? s : __expf(x) - 1.0f;
 }
 template <bool FAST>
 __device__ __forceinline__ float lru_gelu(float z) {   // (1 + tanh w) / 2 = sigmoid(2 w)
@@ -53,8 +74,9 @@ __device__ __forceinline__ float lru_gelu(float z) {   // (1 + tanh w) / 2 = sig
 // (a, b) of S <- a S + b.  Both from e = a - 1, which keeps its digits where a is nearly one: 1 - a^2 = -e (2 + e).
 template <bool FAST>
 __device__ __forceinline__ float2 lru_coefficients(float r_pre, float i_pre, float u, float rate) {
-  const float e = expm1f(rate * lru_sigmoid<FAST>(r_pre));
-  return make_float2(1.0f + e, sqrtf(-e * (2.0f + e)) * lru_sigmoid<FAST>(i_pre) * u);
+  const float la = rate * lru_sigmoid<FAST>(r_pre);
+  const float e = FAST ? lru_quick_expm1(la) : expm1f(la), q = -e * (2.0f + e);
+  return make_float2(1.0f + e, (FAST ? lru_quick_root(q) : sqrtf(q)) * lru_sigmoid<FAST>(i_pre) * u);
 }
 
 // ---------------------------------------------------------------- conv: a thread per (run of tokens, channel)
@@ -101,6 +123,50 @@ __global__ void __launch_bounds__(LRU_CONV_THREADS) lru_conv_kernel(const Lru P)
         acc = fmaf(P.conv_w[(size_t)j * P.width + c], lru_input(P, t, taps - 1 - j, in_step, pos, ring, c), acc);
     }
     P.u[(size_t)t * P.width + c] = acc;
+  }
+}
+
+// The same for taps that stay in registers, four channels a thread (width in multiples of four, aligned).
+template <int TAPS>
+__global__ void __launch_bounds__(LRU_CONV_THREADS) lru_conv_vec_kernel(const Lru P) {
+  pdl_trigger();
+  pdl_wait();
+  const int c = 4 * (blockIdx.y * LRU_CONV_THREADS + threadIdx.x);
+  if (c >= P.width) return;
+  const int t0 = blockIdx.x * LRU_RUN, t1 = min(P.n_tokens, t0 + LRU_RUN);
+  const float4 bias = *reinterpret_cast<const float4*>(P.conv_b + c);
+  float4 w[TAPS], hist[TAPS];
+#pragma unroll
+  for (int j = 0; j < TAPS; j++) {
+    w[j] = *reinterpret_cast<const float4*>(P.conv_w + (size_t)j * P.width + c);
+    hist[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+#pragma unroll
+  for (int i = 0; i < LRU_RUN; i++) {
+    const int t = t0 + i;
+    if (t >= t1) break;
+    const int seq = P.token_seq[t], pos = P.token_pos[t];
+    const int in_step = seq >= 0 ? t - P.seq_start[seq] : 0;
+    if (i == 0 || in_step == 0) {
+      const float* ring = seq >= 0 ? P.state + (size_t)P.seq_slot[seq] * P.state_stride + P.width : nullptr;
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; j++) {
+        const int back = TAPS - 1 - j;
+        if (back <= in_step) hist[j] = ld_fresh((const float4*)(P.x + (size_t)(t - back) * P.ld + c));
+        else if (ring && pos - back >= 0) hist[j] = ld_fresh((const float4*)(ring + (size_t)((pos - back) % TAPS) * P.width + c));
+        else hist[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+    }
+    hist[TAPS - 1] = ld_fresh((const float4*)(P.x + (size_t)t * P.ld + c));
+    float4 u = bias;
+#pragma unroll
+    for (int j = 0; j < TAPS; j++) {                 // oldest input first: the order of the other form
+      u.x = fmaf(w[j].x, hist[j].x, u.x); u.y = fmaf(w[j].y, hist[j].y, u.y);
+      u.z = fmaf(w[j].z, hist[j].z, u.z); u.w = fmaf(w[j].w, hist[j].w, u.w);
+    }
+    *reinterpret_cast<float4*>(P.u + (size_t)t * P.width + c) = u;
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; j++) hist[j] = hist[j + 1];
   }
 }
 
@@ -255,24 +321,40 @@ __global__ void __launch_bounds__(LS_MAX_WARPS * 32, 2) lru_scan_kernel(const Lr
     const int t0 = base + stretch * LS_TOKENS;
     float a[LS_TOKENS], b[LS_TOKENS], yv[LS_TOKENS];
     float uu[LS_TOKENS], rr[LS_TOKENS], ii[LS_TOKENS];
-#pragma unroll
-    for (int j = 0; j < LS_TOKENS; j++) {            // all loads of the stretch first
-      const int t = t0 + j;
-      const bool ok = live && t < r1;
-      uu[j] = ok ? P.u[(size_t)t * P.width + c] : 0.f;
-      rr[j] = ok ? P.pre[(size_t)t * 2 * P.width + col_r] : 0.f;
-      ii[j] = ok ? P.pre[(size_t)t * 2 * P.width + col_i] : 0.f;
-      yv[j] = ok ? P.y[(size_t)t * P.ld + c] : 0.f;
-    }
+    const float* pu = P.u + (size_t)t0 * P.width + cc;
+    const float* pr = P.pre + (size_t)t0 * 2 * P.width + col_r;
+    const float* py = P.y + (size_t)t0 * P.ld + cc;
     float A = 1.f, H = 0.f;
+    if (t0 + LS_TOKENS <= r1) {                      // a whole stretch (channels beyond the width read the first one's)
 #pragma unroll
-    for (int j = 0; j < LS_TOKENS; j++) {
-      const float2 ab = lru_coefficients<FAST>(rr[j] + bias_r, ii[j] + bias_i, uu[j], rate);
-      const bool ok = t0 + j < r1;
-      a[j] = ok ? ab.x : 1.f;
-      b[j] = ok ? ab.y : 0.f;
-      A *= a[j];
-      H = fmaf(a[j], H, b[j]);
+      for (int j = 0; j < LS_TOKENS; j++) {          // all loads of the stretch first
+        uu[j] = pu[(size_t)(j * P.width)];
+        rr[j] = pr[(size_t)(2 * j * P.width)];
+        ii[j] = pr[(size_t)(2 * j * P.width) + size];
+        yv[j] = py[(size_t)j * P.ld];
+      }
+#pragma unroll
+      for (int j = 0; j < LS_TOKENS; j++) {
+        const float2 ab = lru_coefficients<FAST>(rr[j] + bias_r, ii[j] + bias_i, uu[j], rate);
+        a[j] = ab.x;
+        b[j] = ab.y;
+        A *= a[j];
+        H = fmaf(a[j], H, b[j]);
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < LS_TOKENS; j++) {
+        const bool ok = t0 + j < r1;
+        uu[j] = ok ? pu[(size_t)(j * P.width)] : 0.f;
+        rr[j] = ok ? pr[(size_t)(2 * j * P.width)] : 0.f;
+        ii[j] = ok ? pr[(size_t)(2 * j * P.width) + size] : 0.f;
+        yv[j] = ok ? py[(size_t)j * P.ld] : 0.f;
+        const float2 ab = lru_coefficients<FAST>(rr[j] + bias_r, ii[j] + bias_i, uu[j], rate);
+        a[j] = ok ? ab.x : 1.f;
+        b[j] = ok ? ab.y : 0.f;
+        A *= a[j];
+        H = fmaf(a[j], H, b[j]);
+      }
     }
     ends[buf][stretch][lane] = make_float2(A, H);
     __syncthreads();                                 // (the other buffer's readers are past their loop: one barrier a round)
@@ -283,10 +365,11 @@ __global__ void __launch_bounds__(LS_MAX_WARPS * 32, 2) lru_scan_kernel(const Lr
       const float2 e = ends[buf][w][lane];
       S = fmaf(e.x, S, e.y);
     }
+    T* po = (T*)P.out + (size_t)t0 * P.ldo + cc;
 #pragma unroll
     for (int j = 0; j < LS_TOKENS; j++) {
       mine = fmaf(a[j], mine, b[j]);
-      if (live && t0 + j < r1) ((T*)P.out)[(size_t)(t0 + j) * P.ldo + c] = from_float<T>(mine * lru_gelu<FAST>(yv[j]));
+      if (live && t0 + j < r1) po[(size_t)(j * P.ldo)] = from_float<T>(mine * lru_gelu<FAST>(yv[j]));
     }
   }
   if (P.write_state && live && stretch == 0) {
@@ -449,6 +532,15 @@ STRATUM_EXPORT int stratum_lru_conv(const Lru* params, cudaStream_t stream) {
   if (P.n_tokens <= 0) return 0;
   const int bad = lru_check(P);
   if (bad) return bad;
+  const uintptr_t bits = (uintptr_t)P.x | (uintptr_t)P.u | (uintptr_t)P.conv_w | (uintptr_t)P.conv_b | (uintptr_t)P.state;
+  if (P.width % 4 == 0 && P.ld % 4 == 0 && P.state_stride % 4 == 0 && (bits & 15) == 0 && P.taps >= 2 && P.taps <= 4) {
+    const dim3 g4((P.n_tokens + LRU_RUN - 1) / LRU_RUN, (P.width / 4 + LRU_CONV_THREADS - 1) / LRU_CONV_THREADS);
+    if (g4.y > 65535) return STRATUM_ERR_LIMIT;
+    if (P.taps == 2) launch_pdl(lru_conv_vec_kernel<2>, g4, LRU_CONV_THREADS, 0, stream, P);
+    else if (P.taps == 3) launch_pdl(lru_conv_vec_kernel<3>, g4, LRU_CONV_THREADS, 0, stream, P);
+    else launch_pdl(lru_conv_vec_kernel<4>, g4, LRU_CONV_THREADS, 0, stream, P);
+    return launch_status();
+  }
   const dim3 grid((P.n_tokens + LRU_RUN - 1) / LRU_RUN, (P.width + LRU_CONV_THREADS - 1) / LRU_CONV_THREADS);
   if (grid.y > 65535) return STRATUM_ERR_LIMIT;
   switch (P.taps) {

@@ -193,19 +193,31 @@ __global__ void __launch_bounds__(QK_ROW_THREADS) qk_norm_rope_row_kernel(const 
     const float m = P.per_head ? mul[h] : (is_q ? ssq : ssk);
     const float* gain = is_q ? P.q_gain : P.k_gain;
     const int g0 = P.per_head ? d0 : (is_q ? c : c - nq);
-    float out[4];
+    const float4 own = *reinterpret_cast<const float4*>(qk_row + c), og = *reinterpret_cast<const float4*>(gain + g0);
+    float out[4] = {own.x * m * og.x, own.y * m * og.y, own.z * m * og.z, own.w * m * og.w};
+    if (d0 < 2 * rp) {
+      if (P.half) {                                  // (rot_pairs is a multiple of four: four dimensions turn alike)
+        const bool second = d0 >= rp;
+        const int step = second ? -rp : rp, pair = second ? d0 - rp : d0;
+        const float4 w = *reinterpret_cast<const float4*>(qk_row + c + step);
+        const float4 wg = *reinterpret_cast<const float4*>(gain + g0 + step);
+        const float4 f0 = *reinterpret_cast<const float4*>(cs + pair), f1 = *reinterpret_cast<const float4*>(cs + pair + 2);
+        const float mate[4] = {w.x * m * wg.x, w.y * m * wg.y, w.z * m * wg.z, w.w * m * wg.w};
+        const float cc[4] = {f0.x, f0.z, f1.x, f1.z}, ss[4] = {f0.y, f0.w, f1.y, f1.w};
 #pragma unroll
-    for (int i = 0; i < 4; i++) {
-      const int d = d0 + i;
-      float v = qk_row[c + i] * m * gain[g0 + i];
-      if (d < 2 * rp) {
-        const bool second = P.half ? d >= rp : d & 1;
-        const int step = P.half ? (second ? -rp : rp) : (second ? -1 : 1), pair = P.half ? (second ? d - rp : d) : d >> 1;
-        const float w = qk_row[c + i + step] * m * gain[g0 + i + step];
-        const float2 f = cs[pair];
-        v = (second ? v * f.x + w * f.y : v * f.x - w * f.y) * P.magnitude;
+        for (int i = 0; i < 4; i++)
+          out[i] = (second ? out[i] * cc[i] + mate[i] * ss[i] : out[i] * cc[i] - mate[i] * ss[i]) * P.magnitude;
+      } else {
+#pragma unroll
+        for (int i = 0; i < 4; i += 2) {
+          if (d0 + i < 2 * rp) {
+            const float2 f = cs[(d0 + i) >> 1];
+            const float u = out[i], v = out[i + 1];
+            out[i] = (u * f.x - v * f.y) * P.magnitude;
+            out[i + 1] = (v * f.x + u * f.y) * P.magnitude;
+          }
+        }
       }
-      out[i] = v;
     }
     const float4 v4 = make_float4(out[0], out[1], out[2], out[3]);
     if (is_q) {
@@ -228,9 +240,10 @@ STRATUM_EXPORT int stratum_qk_norm_rope(const QKNormRope* params, int dtype, cud
   const size_t smem = P.per_head ? (size_t)(P.n_heads + P.n_kv) * sizeof(float) : 0;
   if (smem > 40 * 1024) return STRATUM_ERR_LIMIT;
   // (which form: by sizes and alignment alone, which a model's buffers share from step to step)
-  const uintptr_t bits = (uintptr_t)P.proj | (uintptr_t)P.q_out | (uintptr_t)P.k_cache | (uintptr_t)P.v_cache;
+  const uintptr_t bits = (uintptr_t)P.proj | (uintptr_t)P.q_out | (uintptr_t)P.k_cache | (uintptr_t)P.v_cache |
+                         (uintptr_t)P.q_gain | (uintptr_t)P.k_gain;
   const size_t row_smem = ((size_t)(P.n_heads + P.n_kv) * (P.dim + 1) + 2 * (size_t)P.rot_pairs) * sizeof(float);
-  if (P.dim % 4 == 0 && P.v_dim % 4 == 0 && P.ld % 4 == 0 && P.ldq % 4 == 0 && (bits & 15) == 0 && row_smem <= 100 * 1024 &&
+  if (P.dim % 4 == 0 && (!P.half || P.rot_pairs % 4 == 0) && P.v_dim % 4 == 0 && P.ld % 4 == 0 && P.ldq % 4 == 0 && (bits & 15) == 0 && row_smem <= 100 * 1024 &&
       (dtype == STRATUM_DT_F32 || dtype == STRATUM_DT_BF16)) {
     void (*kern)(const QKNormRope) = dtype == STRATUM_DT_F32 ? qk_norm_rope_row_kernel<float> : qk_norm_rope_row_kernel<bf16>;
     if (row_smem > 40 * 1024) {

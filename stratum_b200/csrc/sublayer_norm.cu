@@ -104,8 +104,25 @@ __global__ void cast_rows_kernel(const float* x, bf16* out, size_t n) {
   if (i < n) out[i] = __float2bfloat16_rn(ld_fresh(x + i));
 }
 
+__global__ void cast_rows_vec_kernel(const float* x, bf16* out, size_t n4) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n4) return;
+  const float4 v = ld_fresh(reinterpret_cast<const float4*>(x) + i);
+  __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 pk;
+  pk.x = *reinterpret_cast<uint32_t*>(&lo);
+  pk.y = *reinterpret_cast<uint32_t*>(&hi);
+  reinterpret_cast<uint2*>(out)[i] = pk;
+}
+
 STRATUM_EXPORT int stratum_cast_rows(const float* x, void* out, long long n, cudaStream_t stream) {
   if (n <= 0) return 0;
+  if (n % 4 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0 && (n / 4 + 255) / 256 <= 0x7fffffffLL) {
+    launch_pdl(cast_rows_vec_kernel, (unsigned)((n / 4 + 255) / 256), 256, 0, stream, x, (bf16*)out, (size_t)(n / 4));
+    return launch_status();
+  }
   const long long blocks = (n + 255) / 256;
   if (blocks > 0x7fffffffLL) return STRATUM_ERR_LIMIT;
   launch_pdl(cast_rows_kernel, (unsigned)blocks, 256, 0, stream, x, (bf16*)out, (size_t)n);

@@ -43,7 +43,7 @@ __device__ __forceinline__ void sn_axpy(float4& z, float a, float4 y, float4 g) 
 
 // Rows whose groups are a multiple of four values, at most KEEP pieces of four per thread; `team` warps per group.
 // (as many warps as the registers of KEEP pieces leave room for)
-__host__ __device__ constexpr int sn_most_warps(int keep) { return keep == 2 ? 32 : (keep == 4 ? 24 : 16); }
+__host__ __device__ constexpr int sn_most_warps(int keep) { return keep == 2 ? 32 : 16; }
 
 template <typename T, int KEEP>
 __global__ void __launch_bounds__(sn_most_warps(KEEP) * 32) sum_norm_vec_kernel(const SumNorm P, int team) {
@@ -178,9 +178,9 @@ static int launch_sum_norm(const SumNorm& P, cudaStream_t stream) {
   if (size % 4 == 0 && (bits & 15) == 0 && n_groups <= 32) {
     const int pieces = size / 4;
     int keep = 0, team = 0;
-    for (int k = 2; k <= 8 && !keep; k *= 2) {
+    for (int k : {4, 8, 2}) {
       team = (pieces + 32 * k - 1) / (32 * k);
-      if (team * n_groups <= sn_most_warps(k)) keep = k;
+      if (team * n_groups <= sn_most_warps(k)) { keep = k; break; }
     }
     if (keep) {
       const dim3 block(n_groups * team * 32);
