@@ -4,10 +4,12 @@
 //   o_i = c^(i + 1) q_i S + sum over j <= i of c^(i - j) (q_i . k_j) v_j          (times q_scale)
 //   S  <- c^n S + sum_j k_j (c^(n - 1 - j) v_j)^T
 //
-// The state stays in float32 registers from the first chunk to the last.  Every factor of a product is float32 and goes
-// to the tensor cores in two bfloat16 parts (x = hi + lo to 16 bits of mantissa), as hi hi + hi lo + lo hi with float32
-// sums, so a product is as good as its factors' 16 bits; the scores q . k and their decays are float32 between the two
-// products they take part in.
+// The state stays in float32 registers from the first chunk to the last.  q, k and v, which are projections, enter the
+// products in two bfloat16 parts (x = hi + lo to 16 bits of mantissa, where a projection need not have more than
+// bfloat16's 8); everything behind them is as wide as float32: the scores with their decays, the decayed values and the
+// state go to the tensor cores in three parts (24 bits), and all products of parts that reach a float32 sum's last place
+// are formed, with float32 sums: the products of the high parts in one accumulator, the small ones in another, and both
+// joined to what came before by ordinary additions (the tensor cores cut their sums off instead of rounding them).
 //
 // A CTA owns (sequence, head, 32 columns of S).  The next chunk's q, k and v are copied to a staging buffer
 // (cp.async) while one is worked on; a chunk's phases, each a barrier apart: split into parts; scores; outputs from
@@ -38,17 +40,21 @@ __device__ __forceinline__ void gc_ldsm2_t(uint32_t (&b)[2], const bf16* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];"
                : "=r"(b[0]), "=r"(b[1]) : "r"((uint32_t)__cvta_generic_to_shared(p)) : "memory");
 }
-// acc += A B with A and B in two parts each (the product of the two low parts is left out)
-__device__ __forceinline__ void gc_mma3(float (&acc)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4],
-                                        const uint32_t (&bh)[2], const uint32_t (&bl)[2]) {
-  mma16816(acc, ah[0], ah[1], ah[2], ah[3], bh[0], bh[1]);
-  mma16816(acc, ah[0], ah[1], ah[2], ah[3], bl[0], bl[1]);
-  mma16816(acc, al[0], al[1], al[2], al[3], bh[0], bh[1]);
+__device__ __forceinline__ void gc_mma(float (&acc)[4], const uint32_t (&a)[4], const uint32_t (&b)[2]) {
+  mma16816(acc, a[0], a[1], a[2], a[3], b[0], b[1]);
 }
 __device__ __forceinline__ void gc_split2(float x, float y, bf16* hi, bf16* lo) {
   const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
   *reinterpret_cast<__nv_bfloat162*>(hi) = h;
   *reinterpret_cast<uint32_t*>(lo) = pack_bf16(x - __bfloat162float(h.x), y - __bfloat162float(h.y));
+}
+// three parts, `step` values apart: 24 bits of mantissa together
+__device__ __forceinline__ void gc_split3(float x, float y, bf16* p, int step) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+  x -= __bfloat162float(h.x);
+  y -= __bfloat162float(h.y);
+  *reinterpret_cast<__nv_bfloat162*>(p) = h;
+  gc_split2(x, y, p + step, p + 2 * step);
 }
 __device__ __forceinline__ void gc_split4(float4 v, bf16* hi, bf16* lo) {
   gc_split2(v.x, v.y, hi, lo);
@@ -62,7 +68,7 @@ __device__ __forceinline__ void gc_copy16(float* dst_shared, const float* src) {
 // Floats and bfloat16 of shared memory for chunks of C tokens and `dim` key dimensions, in this order.
 __host__ __device__ __forceinline__ size_t gc_smem_bytes(int C, int dim) {
   const size_t floats = (size_t)C * (2 * dim + GC_COLS) + C + 4;                       // staging, powers of the decay
-  const size_t halves = 4 * (size_t)C * (dim + 8) + 2 * (size_t)C * (C + 8) + 4 * (size_t)C * GC_VP + 2 * (size_t)dim * GC_VP;
+  const size_t halves = 4 * (size_t)C * (dim + 8) + 3 * (size_t)C * (C + 8) + 5 * (size_t)C * GC_VP + 3 * (size_t)dim * GC_VP;
   return floats * 4 + halves * 2;
 }
 
@@ -86,14 +92,12 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
   bf16* q_lo = q_hi + C * QP;
   bf16* k_hi = q_lo + C * QP;
   bf16* k_lo = k_hi + C * QP;
-  bf16* a_hi = k_lo + C * QP;                         // [C][AP]
-  bf16* a_lo = a_hi + C * AP;
-  bf16* v_hi = a_lo + C * AP;                         // [C][GC_VP]
-  bf16* v_lo = v_hi + C * GC_VP;
-  bf16* w_hi = v_lo + C * GC_VP;                      // v_j c^(n - 1 - j)
-  bf16* w_lo = w_hi + C * GC_VP;
-  bf16* s_hi = w_lo + C * GC_VP;                      // [D][GC_VP]
-  bf16* s_lo = s_hi + D * GC_VP;
+  const int A1 = C * AP, W1 = C * GC_VP, S1 = D * GC_VP;        // from a part of the scores, values, state to the next
+  bf16* a_p = k_lo + C * QP;                          // [3][C][AP]
+  bf16* v_hi = a_p + 3 * A1;                          // [C][GC_VP]
+  bf16* v_lo = v_hi + W1;
+  bf16* w_p = v_lo + W1;                              // [3][C][GC_VP]: v_j c^(n - 1 - j)
+  bf16* s_p = w_p + 3 * W1;                           // [3][D][GC_VP]
 
   const int seq = blockIdx.z, h = blockIdx.y, j0 = blockIdx.x * GC_COLS;
   const int r0 = P.seq_start[seq], r1 = P.seq_start[seq + 1];
@@ -129,8 +133,8 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
 #pragma unroll
       for (int n = 0; n < NS; n++) {
         const int at = d * GC_VP + scol + 8 * n + 2 * t;
-        gc_split2(S[b][n][0], S[b][n][1], s_hi + at, s_lo + at);
-        gc_split2(S[b][n][2], S[b][n][3], s_hi + at + 8 * GC_VP, s_lo + at + 8 * GC_VP);
+        gc_split3(S[b][n][0], S[b][n][1], s_p + at, S1);
+        gc_split3(S[b][n][2], S[b][n][3], s_p + at + 8 * GC_VP, S1);
       }
     }
   };
@@ -174,7 +178,8 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
         gc_split4(v, v_hi + at, v_lo + at);
         const float w = tok < n_here ? power[n_here - 1 - tok] : 0.f;
         v.x *= w; v.y *= w; v.z *= w; v.w *= w;
-        gc_split4(v, w_hi + at, w_lo + at);
+        gc_split3(v.x, v.y, w_p + at, W1);
+        gc_split3(v.z, v.w, w_p + at + 2, W1);
       }
     }
     __syncthreads();                                  // the parts are there and the staging buffer is free
@@ -182,9 +187,11 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
 
     // ---- scores of 16 tokens against C / CW keys, decayed; what lies ahead of a token is zero
     {
-      float acc[NA][4];
+      float acc[NA][4], rest[NA][4];
 #pragma unroll
-      for (int n = 0; n < NA; n++) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+      for (int n = 0; n < NA; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) acc[n][e] = rest[n][e] = 0.f;
       const int first = cw * NA;                      // this warp's first block of 8 keys
       if (8 * first <= 16 * rb + 15) {
         for (int d = 0; d < D; d += 16) {
@@ -198,7 +205,10 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
             const int bt = (8 * (first + n) + (lane & 7)) * QP + d + 8 * ((lane >> 3) & 1);
             gc_ldsm2(bh, k_hi + bt);
             gc_ldsm2(bl, k_lo + bt);
-            gc_mma3(acc[n], ah, al, bh, bl);
+            gc_mma(acc[n], ah, bh);
+            gc_mma(rest[n], al, bl);
+            gc_mma(rest[n], al, bh);
+            gc_mma(rest[n], ah, bl);
           }
         }
       }
@@ -208,18 +218,20 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
 #pragma unroll
         for (int e = 0; e < 2; e++) {
           const int i = 16 * rb + g + 8 * e;
-          const float x = j <= i ? acc[n][2 * e] * power[i - j] : 0.f;
-          const float y = j + 1 <= i ? acc[n][2 * e + 1] * power[i - j - 1] : 0.f;
-          gc_split2(x, y, a_hi + i * AP + j, a_lo + i * AP + j);
+          const float x = j <= i ? (acc[n][2 * e] + rest[n][2 * e]) * power[i - j] : 0.f;
+          const float y = j + 1 <= i ? (acc[n][2 * e + 1] + rest[n][2 * e + 1]) * power[i - j - 1] : 0.f;
+          gc_split3(x, y, a_p + i * AP + j, A1);
         }
       }
     }
     __syncthreads();
     // ---- outputs of 16 tokens, NO blocks of 8 columns
     {
-      float acc[NO][4];
+      float acc[NO][4], rest[NO][4], sum[NO][4];
 #pragma unroll
-      for (int n = 0; n < NO; n++) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+      for (int n = 0; n < NO; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) acc[n][e] = rest[n][e] = 0.f;
       for (int d = 0; d < D; d += 16) {
         uint32_t ah[4], al[4];
         const int at = (16 * rb + (lane & 15)) * QP + d + 8 * (lane >> 4);
@@ -227,30 +239,45 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
         gc_ldsm4(al, q_lo + at);
 #pragma unroll
         for (int n = 0; n < NO; n++) {
-          uint32_t bh[2], bl[2];
+          uint32_t b0[2], b1[2], b2[2];
           const int bt = (d + (lane & 15)) * GC_VP + 8 * (cw * NO + n);
-          gc_ldsm2_t(bh, s_hi + bt);
-          gc_ldsm2_t(bl, s_lo + bt);
-          gc_mma3(acc[n], ah, al, bh, bl);
+          gc_ldsm2_t(b0, s_p + bt);
+          gc_ldsm2_t(b1, s_p + S1 + bt);
+          gc_ldsm2_t(b2, s_p + 2 * S1 + bt);
+          gc_mma(acc[n], ah, b0);
+          gc_mma(rest[n], ah, b2);
+          gc_mma(rest[n], al, b1);
+          gc_mma(rest[n], ah, b1);
+          gc_mma(rest[n], al, b0);
         }
       }
       const float p0 = power[16 * rb + g + 1], p1 = power[16 * rb + g + 9];
 #pragma unroll
-      for (int n = 0; n < NO; n++) { acc[n][0] *= p0; acc[n][1] *= p0; acc[n][2] *= p1; acc[n][3] *= p1; }
+      for (int n = 0; n < NO; n++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+          sum[n][e] = (acc[n][e] + rest[n][e]) * (e < 2 ? p0 : p1);
+          acc[n][e] = rest[n][e] = 0.f;
+        }
 #pragma unroll
       for (int kb = 0; kb < RB; kb++) {
         if (kb > rb) break;                           // keys ahead of the whole block of tokens
-        uint32_t ah[4], al[4];
+        uint32_t a0[4], a1[4], a2[4];
         const int at = (16 * rb + (lane & 15)) * AP + 16 * kb + 8 * (lane >> 4);
-        gc_ldsm4(ah, a_hi + at);
-        gc_ldsm4(al, a_lo + at);
+        gc_ldsm4(a0, a_p + at);
+        gc_ldsm4(a1, a_p + A1 + at);
+        gc_ldsm4(a2, a_p + 2 * A1 + at);
 #pragma unroll
         for (int n = 0; n < NO; n++) {
           uint32_t bh[2], bl[2];
           const int bt = (16 * kb + (lane & 15)) * GC_VP + 8 * (cw * NO + n);
           gc_ldsm2_t(bh, v_hi + bt);
           gc_ldsm2_t(bl, v_lo + bt);
-          gc_mma3(acc[n], ah, al, bh, bl);
+          gc_mma(acc[n], a0, bh);
+          gc_mma(rest[n], a2, bh);
+          gc_mma(rest[n], a1, bl);
+          gc_mma(rest[n], a1, bh);
+          gc_mma(rest[n], a0, bl);
         }
       }
 #pragma unroll
@@ -262,7 +289,8 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
           const int i = 16 * rb + g + 8 * e;
           if (i < n_here)
             *reinterpret_cast<float2*>(P.o_raw + (size_t)(c0 + i) * HV + (size_t)h * V + j) =
-                make_float2(acc[n][2 * e] * P.q_scale, acc[n][2 * e + 1] * P.q_scale);
+                make_float2((sum[n][2 * e] + (acc[n][2 * e] + rest[n][2 * e])) * P.q_scale,
+                            (sum[n][2 * e + 1] + (acc[n][2 * e + 1] + rest[n][2 * e + 1])) * P.q_scale);
         }
       }
     }
@@ -273,8 +301,11 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
       for (int b = 0; b < MB; b++) {
         const int d0 = 16 * (srow + 8 * b);
         if (d0 >= D) continue;
+        float acc[NS][4], rest[NS][4];
 #pragma unroll
-        for (int n = 0; n < NS; n++) { S[b][n][0] *= pn; S[b][n][1] *= pn; S[b][n][2] *= pn; S[b][n][3] *= pn; }
+        for (int n = 0; n < NS; n++)
+#pragma unroll
+          for (int e = 0; e < 4; e++) acc[n][e] = rest[n][e] = 0.f;
 #pragma unroll
         for (int kb = 0; kb < RB; kb++) {
           uint32_t ah[4], al[4];
@@ -283,13 +314,22 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
           gc_ldsm4_t(al, k_lo + at);
 #pragma unroll
           for (int n = 0; n < NS; n++) {
-            uint32_t bh[2], bl[2];
+            uint32_t b0[2], b1[2], b2[2];
             const int bt = (16 * kb + (lane & 15)) * GC_VP + scol + 8 * n;
-            gc_ldsm2_t(bh, w_hi + bt);
-            gc_ldsm2_t(bl, w_lo + bt);
-            gc_mma3(S[b][n], ah, al, bh, bl);
+            gc_ldsm2_t(b0, w_p + bt);
+            gc_ldsm2_t(b1, w_p + W1 + bt);
+            gc_ldsm2_t(b2, w_p + 2 * W1 + bt);
+            gc_mma(acc[n], ah, b0);
+            gc_mma(rest[n], ah, b2);
+            gc_mma(rest[n], al, b1);
+            gc_mma(rest[n], ah, b1);
+            gc_mma(rest[n], al, b0);
           }
         }
+#pragma unroll
+        for (int n = 0; n < NS; n++)
+#pragma unroll
+          for (int e = 0; e < 4; e++) S[b][n][e] = fmaf(S[b][n][e], pn, acc[n][e] + rest[n][e]);
       }
     }
     __syncthreads();                                  // every warp has read the old state
@@ -311,7 +351,7 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
 template <int C, int MB, int WARPS>
 static int gla_chunked_launch(const Gla& P, cudaStream_t stream) {
   const size_t smem = gc_smem_bytes(C, P.dim);
-  if (smem > 225 * 1024) return STRATUM_ERR_LIMIT;
+  if (smem > 227 * 1024) return STRATUM_ERR_LIMIT;
   cudaError_t e = cudaFuncSetAttribute(gla_chunked_kernel<C, MB, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const dim3 grid((P.vdim + GC_COLS - 1) / GC_COLS, P.n_heads, P.n_seqs);

@@ -177,6 +177,33 @@ def test_retention_kernels(heads, dim, vdim, pairs, long, form):
     assert float(st[:, HD * vdim:].abs().max()) == 0.0                                    # nothing beyond a state
 
 
+@pytest.mark.parametrize("heads,dim,vdim", [(3, 64, 32), (2, 128, 128), (2, 256, 36)])
+def test_chunks_of_retention_are_as_wide_as_float32(heads, dim, vdim):
+    """Projections that two bfloat16 parts hold exactly (16 bits): what is left is the width of scores, decayed values and
+    state.  Read-outs and state in chunks against float64, next to the token-by-token form's own float32 rounding."""
+    from stratum_b200 import kernels as K
+    rng = np.random.default_rng(dim)
+    T, HD, HV = 500, heads * dim, heads * vdim
+    proj = _bf16(rng.standard_normal((T, 2 * HD + 2 * HV))) * (1.0 + 2.0 ** -12)
+    proj = _bf16(proj) + _bf16(proj - _bf16(proj))
+    decay = np.float32([0.997, 0.9990234375, 0.6])[:heads]
+    q, k, v = (proj[:, a:b].reshape(T, heads, -1) for a, b in ((0, HD), (HD, 2 * HD), (2 * HD, 2 * HD + HV)))
+    S, want = np.zeros((heads, dim, vdim)), np.zeros((T, heads, vdim))
+    for t in range(T):
+        S = decay.astype(np.float64)[:, None, None] * S + k[t][:, :, None] * v[t][:, None, :]
+        want[t] = np.einsum("hdv,hd->hv", S, q[t])
+    err = {}
+    for chunked in (False, True):
+        st = torch.zeros(1, HD * vdim, device="cuda")
+        g = K.GlaStep(_dev(proj), heads, dim, vdim, 0, 1.0, 1.0, 1e-5, head_decay=_dev(decay))
+        o = torch.empty(T, HV, device="cuda")
+        g.recur(o, st, torch.zeros(T, dtype=torch.int32, device="cuda"), _i32([0, T]), _i32([0]), True, chunked=chunked)
+        got = o.double().cpu().numpy().reshape(T, heads, vdim)
+        err[chunked] = (np.sqrt(np.mean((got - want) ** 2)) / np.sqrt(np.mean(want ** 2)),
+                        np.max(np.abs(st.double().cpu().numpy().reshape(heads, vdim, dim).transpose(0, 2, 1) - S)) / np.max(np.abs(S)))
+    assert err[True][0] < 2e-6 and err[True][1] < 3e-6, err
+
+
 class _Step:
     """The fields of a step's description that the recurrence reads."""
 
