@@ -122,7 +122,7 @@ __global__ void __launch_bounds__(QK_THREADS) qk_norm_rope_kernel(const QKNormRo
 }
 
 // The form for rows in multiples of four values.
-#define QK_ROW_THREADS 512
+#define QK_ROW_THREADS 256
 __device__ __forceinline__ void qk_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
 __device__ __forceinline__ void qk_store4(bf16* p, float4 v) {
   const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
