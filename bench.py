@@ -519,8 +519,9 @@ def main() -> int:
                     help="layer sizes for the short lines of --decode-only / --prefill-only")
     ap.add_argument("--compare", default=None, choices=["nibelorn", "dabodra", "vitinex", "mokatar", "getizen"],
                     help="instead of the main workload: prefill and decode throughput of the Nibelorn, the Dabodra, "
-                         "the Vitinex or the Mokatar decoder beside a Llama decoder of equal size (Vitinex and Mokatar also beside Dabodra, Getizen beside Mokatar), at 1B-like and 8B-like layer sizes (--layers of "
-                         "them, default 8)")
+                         "the Vitinex, the Mokatar or the Getizen decoder beside a Llama decoder of equal size (Vitinex "
+                         "and Mokatar also beside Dabodra, Getizen beside Mokatar), at 1B-like and 8B-like layer sizes "
+                         "(--layers of them, default 8)")
     ap.add_argument("--kernels", action="store_true",
                     help="with --compare: also the device time of every kernel of one prompt and one decode step")
     ap.add_argument("--prefill-only", action="store_true",

@@ -130,7 +130,7 @@ def test_pages_of_chunks(chunk, step):
 
 def test_rescaled_frequencies():
     from stratum_b200.parts.rope import precise_frequencies
-    for sc in ({"factor": 8.0, "low": 1.0, "high": 4.0, "original": 512}, {"factor": 0.5, "low": 2.0, "high": 3.0, "original": 40},
+    for sc in ({"factor": 6.0, "low": 0.8, "high": 5.0, "original": 700}, {"factor": 0.5, "low": 2.0, "high": 3.0, "original": 40},
                {"factor": 3.0, "low": 2.0, "high": 2.0, "original": 100}):
         rot = {"base": 20000.0, "dims": 48, "scaling": sc}
         got, mag = precise_frequencies(48, 20000.0, {"kind": "llama3", "factor": sc["factor"], "low_freq_factor": sc["low"],

@@ -186,7 +186,7 @@ def test_chunks_of_retention_are_as_wide_as_float32(heads, dim, vdim):
     T, HD, HV = 500, heads * dim, heads * vdim
     proj = _bf16(rng.standard_normal((T, 2 * HD + 2 * HV))) * (1.0 + 2.0 ** -12)
     proj = _bf16(proj) + _bf16(proj - _bf16(proj))
-    decay = np.float32([0.997, 0.9990234375, 0.6])[:heads]
+    decay = np.float32([0.997, 0.9985, 0.6])[:heads]
     q, k, v = (proj[:, a:b].reshape(T, heads, -1) for a, b in ((0, HD), (HD, 2 * HD), (2 * HD, 2 * HD + HV)))
     S, want = np.zeros((heads, dim, vdim)), np.zeros((T, heads, vdim))
     for t in range(T):
