@@ -1,1 +1,1 @@
-from . import dabodra, getizen, llama, mokatar, nibelorn, vitinex  # noqa: F401  (registers the architectures)
+from . import dabodra, getizen, llama, memipel, mokatar, nibelorn, vitinex  # noqa: F401  (registers the architectures)

@@ -12,7 +12,8 @@
 //   a_m        = sum_t softmax_t(score) V_t[vh]           over the keys t in [lo, p], lo = 0 or p - window + 1,
 //                                                         and with a window also the keys t < keep_first;
 //                                                         chunked (mask_chunk): only keys of p's own chunk of positions
-// head_scale: where given, one more factor per head on the score.
+// head_scale: where given, one more factor per head on the score.  slope: where given, slope[h] * (p - t) is taken off the
+//   score (behind the cap, if there is one).
 // Values: rows of the value cache, or (v_in_k) the first v_dim values of the key rows of head (h / group) * maps.
 // sink: where given, exp(sink[h]) is one more term of every softmax's denominator (it has no key and no value).
 // combine 0 (maps = 1): out[h] = a_0, times sigmoid(gate[h * v_dim + d]) element by element where `gate` is given.
@@ -49,6 +50,7 @@ attention_general_kernel(const GeneralAttention P) {
   float temp = 1.f;
   if (P.temp_coef != 0.f) temp = 1.f + P.temp_coef * logf((float)((pos + 1) / P.temp_every) + 1.f);
   const float factor = P.scale * temp * (P.head_scale ? P.head_scale[h] : 1.f);
+  const float slope = P.slope ? P.slope[h] : 0.f;
   const int lo = general_first_key(P, pos);
   // chunks are visited in key order: those that hold kept first keys, then those from the window's first key on
   const int first_win = (lo / 32) * 32;
@@ -92,6 +94,7 @@ attention_general_kernel(const GeneralAttention P) {
         for (int d = 0; d < D; d++) dot = fmaf(qm[d], to_float(kr[d]), dot);
         s = dot * factor;
         if (P.softcap > 0.f) s = P.softcap * tanhf(s / P.softcap);
+        s -= slope * (float)(pos - key);
       }
       const float m_new = fmaxf(m_run[m], warp_max(s));   // finite: every chunk visited holds a valid key
       const float corr = expf(m_run[m] - m_new);          // exp(-inf) = 0 on the first chunk

@@ -19,6 +19,7 @@ struct GeneralAttention {
   const int* seq_start;     // dense keys (tensor-core kernel): first row of every sequence of the step
   const float* sink;        // [n_heads] or null: exp(sink[h]) joins the softmax's denominator (no key, no value, not scaled)
   const float* head_scale;  // [n_heads] or null: a factor on the scores of each head, beside `scale`
+  const float* slope;       // [n_heads] or null: slope[h] * (i - j) is taken off the score of position i against key j
   const float* gate;        // [tokens][ld_gate] or null: pre-activations of an output gate per element (column h * v_dim + d)
   int ldq, ldo, bt_stride, n_tokens;
   int n_heads, group, maps;

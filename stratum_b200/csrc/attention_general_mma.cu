@@ -8,7 +8,7 @@
 //            dimension, Q fragments from shared memory, K fragments straight from the cache rows (a dot product
 //            may visit the dimension in any order as long as Q and K agree: lane t of a row takes the 8
 //            contiguous values 8t..8t+7 of every 32, as attention_mma.cu does);
-//   softmax  scale, query factor, tanh cap and mask in float32; the row maximum of the tile goes through shared
+//   softmax  scale, query factor, tanh cap, distance bias and mask in float32; the row maximum of the tile goes through shared
 //            memory; every warp rescales by the same running maximum and keeps the sum of its own keys;
 //   values   the probabilities are float32; the tensor core takes bfloat16, so each is split into a high and a low
 //            bfloat16 part (p = hi + lo to 16 bits of mantissa) that go through shared memory, and warp w adds
@@ -88,13 +88,14 @@ attention_general_mma_kernel(const GeneralAttention P) {
   // the two rows of this lane in every group of 16 rows: r = g and g + 8;  row -> (token of the group, head)
   int row_tok[RG][2], row_head[2], row_pos[RG][2];
   bool row_ok[RG][2];
-  float row_factor[RG][2];
+  float row_factor[RG][2], row_slope[2];
 #pragma unroll
   for (int e = 0; e < 2; e++) {
     const int r = g + 8 * e;
     const int tr = r / rows_per_token, hr = r % rows_per_token;
     const int hq = hg * 16 + hr;
     row_head[e] = kv * P.group + (hq < P.group ? hq : 0);
+    row_slope[e] = P.slope ? P.slope[row_head[e]] : 0.f;
 #pragma unroll
     for (int rg = 0; rg < RG; rg++) {
       const int tk = rg * tpg + tr;
@@ -226,9 +227,10 @@ attention_general_mma_kernel(const GeneralAttention P) {
           const int e = j >> 1;
           float v = s[rg][i][j] * row_factor[rg][e];
           if (P.softcap > 0.f) v = P.softcap * tanhf(v / P.softcap);
+          const int key = kw + 8 * i + 2 * t + (j & 1);
+          const int pos = row_pos[rg][e];
+          if (P.slope) v -= row_slope[e] * (float)(pos - key);
           if (!whole_tile) {
-            const int key = kw + 8 * i + 2 * t + (j & 1);
-            const int pos = row_pos[rg][e];
             const int lo = lo_of[e];
             const bool ok = any && row_ok[rg][e] && key <= pos && (key >= lo || key < keep) && key < k_end && key >= k_begin;
             v = ok ? v : -INFINITY;

@@ -36,6 +36,8 @@
 // chunks (with `chunk` > 0 a position sees only keys of its own chunk of that many positions) and an output gate (where
 // pre-activations are given, o is multiplied by sigmoid(gate) element by element before it is stored).
 //
+// BIAS (with SPLIT): slope[h] * (p - t) is taken off the scaled score of position p against key t.
+//
 // Every mbarrier wait is bounded (see gemm_tc.cu): on expiry a code goes to the status word and the CTA winds
 // down, freeing its tensor memory.
 #include <math.h>
@@ -55,6 +57,7 @@ struct FaParams {
   bf16* out; int ldo;
   int* status;
   const float* gate; int ld_gate;
+  const float* slope;      // [n_q] or null
   int n_q, n_kv, gs, tokens_per_tile, window, chunk;
   float scale_log2;        // scale * log2(e): exponentials are taken with exp2
 };
@@ -108,7 +111,7 @@ __device__ __forceinline__ FaHalf fa_half(const FaParams& P, int h, int seq, int
   return H;
 }
 
-template <int HD, int NH, bool SPLIT>
+template <int HD, int NH, bool SPLIT, bool BIAS>
 __global__ void __launch_bounds__(FA_THREADS(NH), NH == 1 ? 2 : 1)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, const FaParams P) {
@@ -301,6 +304,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const uint32_t lane_addr = tmem_base + h * 256 + ((uint32_t)(quarter * 32) << 16);
     constexpr int OD = HD / 2;                           // output dims per thread
     const uint32_t o_addr = lane_addr + COL_PV + half * OD;
+    const float slope_log2 = BIAS ? P.slope[kvh * P.gs + head] * 1.4426950408889634f : 0.f;
+    const float to_log2 = BIAS ? 1.0f : P.scale_log2;    // what the (already scaled and shifted) scores still need
     float m_ref = -INFINITY, l = 0.f;                    // reference maximum (scaled, log2 domain); sum of this half
     bool ok = true;
 
@@ -319,6 +324,14 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       // maximum over the whole tile; keys beyond a row's own position (or before its window) are masked, which
       // only tiles on the diagonal (or at the window's edge) need
       const int key0 = (lo_tile + j) * FA_KEYS;
+      if (BIAS) {
+        const float fs = (float)(key0 + half * 32 - pos), ft = (float)(key0 + (half ^ 1) * 32 - pos);
+#pragma unroll
+        for (int i = 0; i < 32; i++) {
+          s[i] = fmaf(s[i], P.scale_log2, slope_log2 * (fs + (float)i));
+          t[i] = fmaf(t[i], P.scale_log2, slope_log2 * (ft + (float)i));
+        }
+      }
       const bool needs_mask = (key0 + FA_KEYS - 1 > H.first_pos) || (SPLIT ? key0 < lo_last : P.window > 0) || (H.ntok < P.tokens_per_tile);
       // (four running maxima, then combined: one chain of 64 dependent comparisons would cost more time than
       // everything else a thread does per tile)
@@ -336,7 +349,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         for (int i = 0; i < 32; i++) mx[i & 3] = max3(mx[i & 3], s[i], t[i]);
       }
       float tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
-      tile_max *= P.scale_log2;                          // scale > 0: the maximum of the scaled scores
+      tile_max *= to_log2;                               // scale > 0: the maximum of the scaled scores
       // the reference moves only when the row's maximum has outgrown it by more than 8 (a factor 256); both
       // threads of a row see the same numbers and decide alike
       const bool grow = tile_max > m_ref + 8.0f;
@@ -348,8 +361,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       float sum0 = 0.f, sum1 = 0.f;
 #pragma unroll
       for (int i = 0; i < 32; i += 2) {
-        const float p0 = fast_exp2(fmaf(s[i], P.scale_log2, -m_use));
-        const float p1 = fast_exp2(fmaf(s[i + 1], P.scale_log2, -m_use));
+        const float p0 = fast_exp2(fmaf(s[i], to_log2, -m_use));
+        const float p1 = fast_exp2(fmaf(s[i + 1], to_log2, -m_use));
         // to bfloat16 by dropping the low mantissa bits (one byte permute for two values; the conversion
         // instruction shares the exponential's pipe, which is the busiest one here).  The probabilities are
         // positive, so every one comes out low by a factor in (1 - 2^-7, 1]; the sums below run over the same
@@ -477,11 +490,11 @@ static int make_map_nd(CUtensorMap* map, const void* base, int rank, const cuuin
   return r == CUDA_SUCCESS ? 0 : STRATUM_ERR_SHAPE;
 }
 
-template <int HD, int NH, bool SPLIT>
+template <int HD, int NH, bool SPLIT, bool BIAS = false>
 static int launch_attention_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const FaParams& P,
                                int n_qblocks, cudaStream_t stream) {
   const size_t smem = sizeof(FaSmem<HD, NH, SPLIT>);
-  auto kern = attention_tc_kernel<HD, NH, SPLIT>;
+  auto kern = attention_tc_kernel<HD, NH, SPLIT, BIAS>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -495,18 +508,19 @@ static int launch_attention_tc(const CUtensorMap& mq, const CUtensorMap& mk, con
 // k_cache / v_cache: bf16 [n_pages][n_kv][64][head_dim].  Query tiles (qb_*): runs of at most
 // halves * 128 / (n_q / n_kv) consecutive new tokens of one sequence (halves: 1 or 2, see the top of this file).
 // head_dim 64 or 128; 128 % (n_q / n_kv) == 0; pages of 64 tokens.  split, chunk, gate (float32 [tokens][ld_gate], n_q *
-// head_dim columns, or null): see the top of this file; split goes with halves = 2.
+// head_dim columns, or null), slope (float32 [n_q], or null): see the top of this file; split goes with halves = 2.
 STRATUM_EXPORT int stratum_attention_tc(const void* q, int ldq, const void* k_cache, const void* v_cache,
                                         long long n_pages, const int* token_pos, const int* block_table,
                                         int bt_stride, const int* qb_seq, const int* qb_tok0, const int* qb_ntok,
                                         int n_qblocks, void* out, int ldo, int n_tokens, int n_q, int n_kv,
                                         int head_dim, int page_tokens, int window, float scale, int halves, int split,
-                                        int chunk, const float* gate, int ld_gate, int* status, cudaStream_t stream) {
+                                        int chunk, const float* gate, int ld_gate, const float* slope, int* status,
+                                        cudaStream_t stream) {
   if (n_tokens <= 0 || n_qblocks <= 0) return 0;
   if (halves != 1 && halves != 2) return STRATUM_ERR_SHAPE;
   if (head_dim != 64 && head_dim != 128) return STRATUM_ERR_SHAPE;
   if (chunk < 0 || window < 0 || (split && halves != 2) || !(scale > 0.f)) return STRATUM_ERR_SHAPE;
-  if ((gate || chunk) && !split) return STRATUM_ERR_SHAPE;
+  if ((gate || chunk || slope) && !split) return STRATUM_ERR_SHAPE;
   if (gate && (ld_gate < n_q * head_dim || ld_gate % 4 != 0 || ((uintptr_t)gate & 15) != 0)) return STRATUM_ERR_ALIGN;
   if (n_kv < 1 || n_q % n_kv != 0 || page_tokens != FA_KEYS) return STRATUM_ERR_SHAPE;
   const int gs = n_q / n_kv;
@@ -535,8 +549,12 @@ STRATUM_EXPORT int stratum_attention_tc(const void* q, int ldq, const void* k_ca
   P.qb_seq = qb_seq; P.qb_tok0 = qb_tok0; P.qb_ntok = qb_ntok;
   P.out = (bf16*)out; P.ldo = ldo; P.status = status;
   P.n_q = n_q; P.n_kv = n_kv; P.gs = gs; P.tokens_per_tile = R; P.window = window;
-  P.chunk = chunk; P.gate = gate; P.ld_gate = ld_gate;
+  P.chunk = chunk; P.gate = gate; P.ld_gate = ld_gate; P.slope = slope;
   P.scale_log2 = scale * 1.4426950408889634f;
+  if (split && slope) {
+    if (head_dim == 64) return launch_attention_tc<64, 2, true, true>(mq, mk, mv, P, n_qblocks, stream);
+    return launch_attention_tc<128, 2, true, true>(mq, mk, mv, P, n_qblocks, stream);
+  }
   if (split) {
     if (head_dim == 64) return launch_attention_tc<64, 2, true>(mq, mk, mv, P, n_qblocks, stream);
     return launch_attention_tc<128, 2, true>(mq, mk, mv, P, n_qblocks, stream);

@@ -56,7 +56,9 @@ __device__ __forceinline__ float block_sum(float v, float* scratch /* >= 33 floa
 // 1 the exact GELU z * 0.5 * (1 + erf(z / sqrt 2)),  2 its tanh form 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))),
 // 3 the square of relu, max(z, 0)^2.  The gated epilogue (3: pairs of gate and up) takes the same codes for the
 // gate's activation, with 0 standing for silu there, and one more that acts on both: 4 the clamped gate
-// g sigmoid(1.702 g) (u + 1) with g = min(gate, limit) and u = up clamped to [-limit, limit].
+// g sigmoid(1.702 g) (u + 1) with g = min(gate, limit) and u = up clamped to [-limit, limit].  A product whose pairs do
+// not all have one limit (stacked feed-forwards of different constants) names a second one and the output column it
+// holds from (GateLimit).
 #define STRATUM_ACT_NONE 0
 #define STRATUM_ACT_GELU_ERF 1
 #define STRATUM_ACT_GELU_TANH 2
@@ -80,6 +82,12 @@ __device__ __forceinline__ float gated(float gate, float up, int act, float limi
   if (act) return activate(gate, act) * up;
   return gate / (1.0f + (FAST ? __expf(-gate) : expf(-gate))) * up;
 }
+
+struct GateLimit {
+  float limit, beyond;      // `beyond` from output column `first` on, where `first` > 0
+  int first;
+  __device__ __forceinline__ float at(int pair) const { return first > 0 && pair >= first ? beyond : limit; }
+};
 
 // ---------------------------------------------------------------- programmatic dependent launch
 // A kernel launched with launch_pdl may begin while the kernel before it in the stream is still

@@ -467,19 +467,20 @@ STRATUM_EXPORT int stratum_gelu(void* x, int dtype, int n_rows, int width, int l
 // gu holds gate and up interleaved: gu[r][2j] = g_j, gu[r][2j+1] = u_j.
 template <typename T>
 __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int inter, size_t total, int act,
-                              float act_limit) {
+                              GateLimit act_limit) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= total) return;
   const size_t r = i / inter;
   const int j = (int)(i - r * inter);
   const T* p = gu + r * (size_t)(2 * inter) + 2 * j;
   const float g = to_float(p[0]), u = to_float(p[1]);
-  out[i] = from_float<T>(gated<false>(g, u, act, act_limit));      // act: the gate's, 0 = silu
+  out[i] = from_float<T>(gated<false>(g, u, act, act_limit.at(j)));      // act: the gate's, 0 = silu
 }
 
 STRATUM_EXPORT int stratum_swiglu(const void* gu, void* out, int dtype, int n_rows, int inter, int act,
-                                  float act_limit, cudaStream_t stream) {
+                                  float limit, int limit_first, float limit_beyond, cudaStream_t stream) {
   const size_t total = (size_t)n_rows * inter;
+  const GateLimit act_limit = {limit, limit_beyond, limit_first};
   if (total == 0) return 0;
   const int threads = 256;
   const unsigned blocks = (unsigned)((total + threads - 1) / threads);

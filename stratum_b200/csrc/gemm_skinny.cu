@@ -47,7 +47,7 @@ template <int MT, int RT, int EPI>
 __global__ void __launch_bounds__(SK_WARPS * 32)
 gemm_skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, const float* __restrict__ bias,
                    void* __restrict__ out, int M, int N, int K, int ldx, int ldo, int groups_per_block, int act,
-                   float act_limit) {
+                   GateLimit act_limit) {
   constexpr int KS = SK_WARPS / RT;                 // K parts
   __shared__ float part[RT][KS][MT * 8][16 + 1];    // [row tile][k part][x row][weight row]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -163,7 +163,7 @@ gemm_skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, const
       // the unfused path rounds gate and up to bfloat16 before the activation; do the same
       gate = __bfloat162float(__float2bfloat16_rn(gate));
       up = __bfloat162float(__float2bfloat16_rn(up));
-      ((bf16*)out)[(size_t)m * ldo + (n >> 1)] = __float2bfloat16_rn(gated<false>(gate, up, act, act_limit));
+      ((bf16*)out)[(size_t)m * ldo + (n >> 1)] = __float2bfloat16_rn(gated<false>(gate, up, act, act_limit.at(n >> 1)));
     }
   }
   __syncthreads();          // the partial sums are reused by the next group
@@ -183,7 +183,7 @@ static int sm_count() {
 
 template <int MT, int RT, int EPI>
 static int launch_skinny_epi(const bf16* x, const bf16* w, const float* bias, void* out, int M, int N, int K,
-                             int ldx, int ldo, int act, float act_limit, cudaStream_t stream) {
+                             int ldx, int ldo, int act, GateLimit act_limit, cudaStream_t stream) {
   auto kern = gemm_skinny_kernel<MT, RT, EPI>;
   static int resident = 0;                 // blocks of this kernel the whole GPU holds at once
   if (!resident) {
@@ -201,7 +201,7 @@ static int launch_skinny_epi(const bf16* x, const bf16* w, const float* bias, vo
 
 template <int MT, int RT>
 static int launch_skinny(const bf16* x, const bf16* w, const float* bias, void* out, int epilogue, int M, int N,
-                         int K, int ldx, int ldo, int act, float act_limit, cudaStream_t stream) {
+                         int K, int ldx, int ldo, int act, GateLimit act_limit, cudaStream_t stream) {
   switch (epilogue) {
     case 0: return launch_skinny_epi<MT, RT, 0>(x, w, bias, out, M, N, K, ldx, ldo, act, act_limit, stream);
     case 1: return launch_skinny_epi<MT, RT, 1>(x, w, bias, out, M, N, K, ldx, ldo, act, act_limit, stream);
@@ -213,10 +213,11 @@ static int launch_skinny(const bf16* x, const bf16* w, const float* bias, void* 
 
 // x: bf16 [M][ldx], w: bf16 [N][K], bias float32 [N] or null, out [M][ldo] (for SwiGLU: [M][N/2]).
 // Needs K % 8 == 0, ldx % 8 == 0 and 16-byte aligned x and w (checked); M <= 32.
-// act (epilogue 0): an activation applied to what is stored; (epilogue 3): the gate's, with act_limit; see common.cuh.
+// act (epilogue 0): an activation applied to what is stored; (epilogue 3): the gate's, with its limits; see common.cuh.
 STRATUM_EXPORT int stratum_gemm_skinny(const void* x, const void* w, const float* bias, void* out, int epilogue,
-                                       int M, int N, int K, int ldx, int ldo, int act, float act_limit,
-                                       cudaStream_t stream) {
+                                       int M, int N, int K, int ldx, int ldo, int act, float limit,
+                                       int limit_first, float limit_beyond, cudaStream_t stream) {
+  const GateLimit act_limit = {limit, limit_beyond, limit_first};
   if (M <= 0 || N <= 0) return 0;
   if (act != 0 && epilogue != 0 && epilogue != 3) return STRATUM_ERR_SHAPE;
   if (M > 32) return STRATUM_ERR_LIMIT;

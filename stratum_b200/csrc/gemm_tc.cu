@@ -56,7 +56,7 @@ struct EpiExtra {
   int emit_ldx, emit_ld;
   int rope_pairs, bt_stride, n_q, n_kv, head_dim, page_tokens, write_cache;
   int act;            // epilogue 0: an activation applied to what is stored; epilogue 3: the gate's (common.cuh)
-  float act_limit;    // the clamped gate's limit
+  GateLimit act_limit;    // the clamped gate's
 };
 
 __device__ __forceinline__ float epi_row_scale(const EpiExtra& X, int m) {
@@ -183,7 +183,7 @@ __device__ __forceinline__ void tc_store_chunk(const TcParams& P, int m, int col
       for (int e = 0; e < 2; e++) {
         const float gate = __bfloat162float(__float2bfloat16_rn(v[j + 2 * e]));
         const float up = __bfloat162float(__float2bfloat16_rn(v[j + 2 * e + 1]));
-        a[e] = gated<true>(gate, up, P.X.act, P.X.act_limit);
+        a[e] = gated<true>(gate, up, P.X.act, P.X.act_limit.at((col0 + j + 2 * e) >> 1));
       }
       __nv_bfloat162 pr = __floats2bfloat162_rn(a[0], a[1]);
       packed[j / 4] = *reinterpret_cast<uint32_t*>(&pr);
@@ -285,7 +285,7 @@ __device__ __forceinline__ void fixup_store(const PT& P, int m, int n, float4 v)
     for (int j = 0; j < 4; j += 2) {
       if (n + j + 1 < P.N) {
         const float g = __bfloat162float(__float2bfloat16_rn(e[j])), u = __bfloat162float(__float2bfloat16_rn(e[j + 1]));
-        o[j >> 1] = __float2bfloat16_rn(gated<true>(g, u, P.X.act, P.X.act_limit));
+        o[j >> 1] = __float2bfloat16_rn(gated<true>(g, u, P.X.act, P.X.act_limit.at((n + j) >> 1)));
       }
     }
     return;
@@ -828,7 +828,7 @@ __device__ __forceinline__ void sk_store(const SkParams& P, const SkTables& T, i
       val = __bfloat162float(__float2bfloat16_rn(val));
       const float other = __shfl_xor_sync(0xffffffffu, val, 1);     // gate (even n) <-> up (odd n)
       if (m < P.M && n + 1 < P.N && (n & 1) == 0)
-        ((bf16*)P.out)[(size_t)m * P.ldo + (n >> 1)] = __float2bfloat16_rn(gated<true>(val, other, P.X.act, P.X.act_limit));
+        ((bf16*)P.out)[(size_t)m * P.ldo + (n >> 1)] = __float2bfloat16_rn(gated<true>(val, other, P.X.act, P.X.act_limit.at(n >> 1)));
     } else if (m < P.M && n < P.N) {
       const size_t idx = (size_t)m * P.ldo + n;
       if (EPI == 0) ((bf16*)P.out)[idx] = __float2bfloat16_rn(activate(val, P.X.act));

@@ -1,5 +1,6 @@
 // Gated linear attention: a recurrent mixer whose state is one matrix S [dim][vdim] per head, in float32, with a decay
-// per key channel; and retention, the same recurrence with one constant decay per head.
+// per key channel; retention, the same recurrence with one constant decay per head; and lightning attention, retention
+// on q, k and v taken through silu.
 //
 // Per token, from the float32 sums of the fused input projection (row = [q | k | v | g | a]: n_heads * dim twice,
 // n_heads * vdim twice, then `rank` values of the decay's inner projection):
@@ -13,7 +14,8 @@
 // With a constant decay per head (`head_decay`) there is no inner projection and neither cast nor decay; instead
 //   rotate    turns the first dimensions of every head of q and k, in place, by the step's table of cosines and sines,
 //             in pairs (i, i + pairs) or, interleaved, (2i, 2i + 1);
-// and the heads' norm may have no gain.  All of it is float32 whatever the compute dtype.
+// and the heads' norm may have no gain.  `silu_qkv` takes q, k and v through silu where the recurrence reads them, and
+// `norm_all` norms the heads' read-outs together, o / sqrt(mean over all heads(o^2) + eps) * gain * sigmoid(g).  All of it is float32 whatever the compute dtype.
 //
 // The recurrence is sequential in the tokens of a sequence and independent across sequences, heads and columns of S:
 // a block owns (sequence, head, a tile of columns), a lane 16 rows of one column, so a column's read-out is split over
@@ -168,6 +170,20 @@ __global__ void __launch_bounds__(GLA_THREADS) gla_recur_kernel(const Gla P) {
     __syncthreads();                                 // this chunk has landed, and the other buffer is free again
     if (c0 + CHUNK < r1) stage(buf ^ 1, c0 + CHUNK);
     const int n_here = min(CHUNK, r1 - c0);
+    if (P.silu_qkv) {                                // (dimensions beyond dim stay zero)
+      for (int i = threadIdx.x; i < n_here * 2 * KQ; i += GLA_THREADS) {
+        const int tok = i / (2 * KQ), e = i - tok * 2 * KQ;
+        if (e % PITCH < ROWS) {
+          float* p = &kqa_s[buf][tok][0][0] + e;
+          *p = gla_silu(*p);
+        }
+      }
+      for (int i = threadIdx.x; i < n_here * COLS; i += GLA_THREADS) {
+        float* p = &v_s[buf][0][0] + i;
+        *p = gla_silu(*p);
+      }
+      __syncthreads();
+    }
     float* o_row = P.o_raw + (size_t)c0 * HV + (size_t)h * V + (live ? j : 0);
 #pragma unroll 2
     for (int tok = 0; tok < n_here; tok++, o_row += HV) {
@@ -237,6 +253,51 @@ __global__ void __launch_bounds__(128) gla_finish_kernel(const Gla P) {
     out[d] = from_float<T>(ld_fresh(o + d) * mul * (P.gain ? P.gain[d] : 1.0f) * gla_silu(ld_fresh(g + d)));
 }
 
+// One block per token: the norm over all heads together, sigmoid gates.  vec: four values at a time.
+#define GLA_FINISH_THREADS 256
+template <typename T>
+__global__ void __launch_bounds__(GLA_FINISH_THREADS) gla_finish_all_kernel(const Gla P, int vec) {
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();                // o_raw and the projection are the work of kernels before this one: ld_fresh
+  const int t = blockIdx.x, HD = P.n_heads * P.dim, HV = P.n_heads * P.vdim;
+  const float* o = P.o_raw + (size_t)t * HV;
+  const float* g = P.proj + (size_t)t * P.ld + 2 * (size_t)HD + HV;
+  T* out = (T*)P.out + (size_t)t * P.ldo;
+  float ss = 0.f;
+  if (vec) {
+    for (int c = 4 * threadIdx.x; c < HV; c += 4 * GLA_FINISH_THREADS) {
+      const float4 x = ld_fresh(reinterpret_cast<const float4*>(o + c));
+      ss += fmaf(x.w, x.w, fmaf(x.z, x.z, fmaf(x.y, x.y, x.x * x.x)));
+    }
+  } else {
+    for (int c = threadIdx.x; c < HV; c += GLA_FINISH_THREADS) {
+      const float x = ld_fresh(o + c);
+      ss = fmaf(x, x, ss);
+    }
+  }
+  ss = block_sum(ss, scratch);
+  const float mul = 1.0f / sqrtf(ss / (float)HV + P.eps);
+  auto value = [&](float x, float gain, float z) { return x * mul * gain / (1.0f + expf(-z)); };
+  if (vec) {
+    for (int c = 4 * threadIdx.x; c < HV; c += 4 * GLA_FINISH_THREADS) {
+      const float4 x = ld_fresh(reinterpret_cast<const float4*>(o + c)), z = ld_fresh(reinterpret_cast<const float4*>(g + c));
+      const float4 w = P.gain ? *reinterpret_cast<const float4*>(P.gain + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+      const float r[4] = {value(x.x, w.x, z.x), value(x.y, w.y, z.y), value(x.z, w.z, z.z), value(x.w, w.w, z.w)};
+      if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(out + c) = make_float4(r[0], r[1], r[2], r[3]);
+      } else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(r[0], r[1]), hi = __floats2bfloat162_rn(r[2], r[3]);
+        *reinterpret_cast<uint2*>(out + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo),
+                                                        *reinterpret_cast<const uint32_t*>(&hi));
+      }
+    }
+  } else {
+    for (int c = threadIdx.x; c < HV; c += GLA_FINISH_THREADS)
+      out[c] = from_float<T>(value(ld_fresh(o + c), P.gain ? P.gain[c] : 1.0f, ld_fresh(g + c)));
+  }
+}
+
 static unsigned gla_blocks(size_t n) {
   const size_t blocks = (n + 255) / 256;
   return (unsigned)(blocks > 148 * 16 ? 148 * 16 : blocks);
@@ -303,6 +364,16 @@ STRATUM_EXPORT int stratum_gla(const Gla* params, int which, int dtype, cudaStre
     return launch_status();
   }
   if (which != 2) return STRATUM_ERR_SHAPE;
+  if (P.norm_all) {
+    const int elem = dtype == STRATUM_DT_F32 ? 4 : 2;
+    const int vec = P.vdim % 4 == 0 && (P.n_heads * P.dim) % 2 == 0 && P.ld % 4 == 0 && (P.ldo * elem) % 16 == 0 &&
+                    (((uintptr_t)P.proj | (uintptr_t)P.o_raw | (uintptr_t)P.out | (uintptr_t)P.gain) & 15) == 0;
+    if (dtype == STRATUM_DT_F32)
+      launch_pdl(gla_finish_all_kernel<float>, (unsigned)P.n_tokens, GLA_FINISH_THREADS, 0, stream, P, vec);
+    else
+      launch_pdl(gla_finish_all_kernel<bf16>, (unsigned)P.n_tokens, GLA_FINISH_THREADS, 0, stream, P, vec);
+    return launch_status();
+  }
   const long long items = (long long)P.n_tokens * P.n_heads;
   const long long blocks = (items + 3) / 4;
   if (blocks > 0x7fffffffLL) return STRATUM_ERR_LIMIT;

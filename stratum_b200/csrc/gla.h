@@ -1,4 +1,4 @@
-// What the kernels of gated linear attention and retention are told (mirrored field by field by kernels.py: pointers
+// What the kernels of gated linear attention, retention and lightning attention are told (mirrored field by field by kernels.py: pointers
 // first, then 4-byte fields).  See gla.cu for the meaning of every field.
 #pragma once
 #include "common.cuh"
@@ -9,7 +9,7 @@ struct Gla {
   const float* proj;        // [tokens][ld]
   void* inner;              // [tokens][ld_inner], the compute dtype: the decay's inner projection (cast)
   const float* head_decay;  // [n_heads] or null: the decays are alpha's
-  const float* gain;        // [vdim] or null: none
+  const float* gain;        // [vdim] ([n_heads * vdim] with norm_all), or null: none
   float* alpha;             // [tokens][n_heads * dim]: z when `decay` begins, alpha when it ends
   float* o_raw;             // [tokens][n_heads * vdim]
   void* out;                // [tokens][ldo] compute dtype
@@ -20,7 +20,9 @@ struct Gla {
   int ld, ldo, n_tokens, n_seqs;
   int n_heads, dim, vdim, rank;
   int state_stride, write_state, ld_inner, rot_pairs;
-  float eps, inv_tau, q_scale, reserved;
+  float eps, inv_tau, q_scale;
+  int silu_qkv;             // q, k and v are taken through silu when they are read
+  int norm_all;             // finish: one norm over all heads together, gated by sigmoid(g) (0: a norm per head, silu(g))
 };
 
 static int gla_check(const Gla& P) {

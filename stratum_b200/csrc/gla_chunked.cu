@@ -9,7 +9,8 @@
 // bfloat16's 8); everything behind them is as wide as float32: the scores with their decays, the decayed values and the
 // state go to the tensor cores in three parts (24 bits), and all products of parts that reach a float32 sum's last place
 // are formed, with float32 sums: the products of the high parts in one accumulator, the small ones in another, and both
-// joined to what came before by ordinary additions (the tensor cores cut their sums off instead of rounding them).
+// joined to what came before by ordinary additions (the tensor cores cut their sums off instead of rounding them).  With
+// `silu_qkv` q, k and v are taken through silu before they are split.
 //
 // A CTA owns (sequence, head, 32 columns of S).  The next chunk's q, k and v are copied to a staging buffer
 // (cp.async) while one is worked on; a chunk's phases, each a barrier apart: split into parts; scores; outputs from
@@ -65,6 +66,9 @@ __device__ __forceinline__ void gc_copy16(float* dst_shared, const float* src) {
                : "memory");
 }
 
+__device__ __forceinline__ float gc_silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+__device__ __forceinline__ float4 gc_silu(float4 v) { return make_float4(gc_silu(v.x), gc_silu(v.y), gc_silu(v.z), gc_silu(v.w)); }
+
 // Floats and bfloat16 of shared memory for chunks of C tokens and `dim` key dimensions, in this order.
 __host__ __device__ __forceinline__ size_t gc_smem_bytes(int C, int dim) {
   const size_t floats = (size_t)C * (2 * dim + GC_COLS) + C + 4;                       // staging, powers of the decay
@@ -74,7 +78,7 @@ __host__ __device__ __forceinline__ size_t gc_smem_bytes(int C, int dim) {
 
 // C: tokens of a chunk (64 or 32).  MB: blocks of 16 rows of S a warp holds (dim <= 128 MB): eight warps cover the rows, and
 // with sixteen the other eight take the other half of the columns.
-template <int C, int MB, int WARPS>
+template <int C, int MB, int WARPS, bool SILU>
 __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
   extern __shared__ __align__(16) float gc_smem[];
   constexpr int RB = C / 16;                          // blocks of 16 tokens
@@ -169,12 +173,15 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
     {
       for (int tok = warp; tok < C; tok += WARPS)
        for (int d = 4 * lane; d < D; d += 128) {
-        gc_split4(*reinterpret_cast<const float4*>(stage_q + tok * D + d), q_hi + tok * QP + d, q_lo + tok * QP + d);
-        gc_split4(*reinterpret_cast<const float4*>(stage_k + tok * D + d), k_hi + tok * QP + d, k_lo + tok * QP + d);
+        float4 q = *reinterpret_cast<const float4*>(stage_q + tok * D + d), k = *reinterpret_cast<const float4*>(stage_k + tok * D + d);
+        if (SILU) { q = gc_silu(q); k = gc_silu(k); }
+        gc_split4(q, q_hi + tok * QP + d, q_lo + tok * QP + d);
+        gc_split4(k, k_hi + tok * QP + d, k_lo + tok * QP + d);
       }
       for (int i = threadIdx.x; i < C * (GC_COLS / 4); i += blockDim.x) {
         const int tok = i / (GC_COLS / 4), j = 4 * (i % (GC_COLS / 4)), at = tok * GC_VP + j;
         float4 v = *reinterpret_cast<const float4*>(stage_v + tok * GC_COLS + j);
+        if (SILU) v = gc_silu(v);
         gc_split4(v, v_hi + at, v_lo + at);
         const float w = tok < n_here ? power[n_here - 1 - tok] : 0.f;
         v.x *= w; v.y *= w; v.z *= w; v.w *= w;
@@ -348,14 +355,14 @@ __global__ void __launch_bounds__(WARPS * 32) gla_chunked_kernel(const Gla P) {
   }
 }
 
-template <int C, int MB, int WARPS>
+template <int C, int MB, int WARPS, bool SILU>
 static int gla_chunked_launch(const Gla& P, cudaStream_t stream) {
   const size_t smem = gc_smem_bytes(C, P.dim);
   if (smem > 227 * 1024) return STRATUM_ERR_LIMIT;
-  cudaError_t e = cudaFuncSetAttribute(gla_chunked_kernel<C, MB, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  cudaError_t e = cudaFuncSetAttribute(gla_chunked_kernel<C, MB, WARPS, SILU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   const dim3 grid((P.vdim + GC_COLS - 1) / GC_COLS, P.n_heads, P.n_seqs);
-  gla_chunked_kernel<C, MB, WARPS><<<grid, WARPS * 32, smem, stream>>>(P);
+  gla_chunked_kernel<C, MB, WARPS, SILU><<<grid, WARPS * 32, smem, stream>>>(P);
   return launch_status();
 }
 
@@ -368,7 +375,7 @@ STRATUM_EXPORT int stratum_gla_chunked(const Gla* params, cudaStream_t stream) {
   if (bad) return bad;
   if (!P.head_decay || P.dim % 16 != 0 || P.vdim % 4 != 0 || P.ld % 4 != 0) return STRATUM_ERR_SHAPE;
   if (((uintptr_t)P.proj & 15) != 0 || ((uintptr_t)P.o_raw & 7) != 0) return STRATUM_ERR_ALIGN;
-  if (P.dim <= 128) return gla_chunked_launch<64, 1, 16>(P, stream);
-  if (P.dim <= 256) return gla_chunked_launch<32, 2, 8>(P, stream);
+  if (P.dim <= 128) return P.silu_qkv ? gla_chunked_launch<64, 1, 16, true>(P, stream) : gla_chunked_launch<64, 1, 16, false>(P, stream);
+  if (P.dim <= 256) return P.silu_qkv ? gla_chunked_launch<32, 2, 8, true>(P, stream) : gla_chunked_launch<32, 2, 8, false>(P, stream);
   return STRATUM_ERR_LIMIT;
 }

@@ -2,7 +2,7 @@
 //
 // route: per token, z = W_r h (h in the compute dtype, W_r and the sums float32); s = sigmoid(z); the choice score of
 //   expert e is c_e = s_e + correction_e.  The experts form `n_groups` equal groups of neighbours; a group's score is
-//   the sum of its two largest c (of its only c when a group is one expert); only the `keep` best groups stay (the
+//   the sum of its two largest c (of its only c when a group is one expert), or, with group_score = 1, its largest c; only the `keep` best groups stay (the
 //   others' c count as -inf).  The `top` experts with the largest c are chosen (among equals the lowest index), and
 //   their weights are s_e / (sum of the chosen s + 1e-20) * scale.  Written: the chosen experts and their weights
 //   [tokens][top], and the same as a row of n_experts weights with zeros for the others.
@@ -32,7 +32,8 @@ struct MoeRoute {
   float* weights;           // [tokens][top]
   int ldx, ldd, n_tokens, width;
   int n_experts, top, n_groups, keep;
-  float scale, reserved;
+  float scale;
+  int group_score;          // 0: the sum of a group's two largest choice scores, 1: the largest
   const float* w_gate;      // [width] or null
   int score, renorm;        // score: 0 sigmoid, 1 softmax over all experts;  renorm: weights divided by their sum
   const float* bias;        // [n_experts] or null: added to the logits z before anything else
@@ -139,7 +140,7 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(const MoeRoute
       const float v = c[g * per + i];
       if (v > a) { b = a; a = v; } else if (v > b) b = v;
     }
-    gs[g] = per > 1 ? a + b : a;
+    gs[g] = per > 1 && P.group_score == 0 ? a + b : a;
   }
   __syncwarp();
   if (P.keep < G) {

@@ -287,13 +287,21 @@ def gelu(x: torch.Tensor, kind: int = GELU_ERF) -> None:
     _check(f(_ptr(x), dtype_code(x.dtype), x.shape[0], x.shape[1], x.stride(0), kind, _stream()), "gelu")
 
 
-def swiglu(gu: torch.Tensor, out: torch.Tensor, act: int = 0, limit: float = 0.0) -> None:
+def _limits(limit):
+    """A clamped gate's limit as the kernels take it, (limit, first, beyond): a number, or such a triple (`beyond` holds
+    from output column `first` on)."""
+    return (float(limit), 0, 0.0) if not isinstance(limit, tuple) else (float(limit[0]), int(limit[1]), float(limit[2]))
+
+
+def swiglu(gu: torch.Tensor, out: torch.Tensor, act: int = 0, limit=0.0) -> None:
     """out[r][j] = silu(gu[r][2j]) * gu[r][2j+1]; with act (ACT_*), that activation takes silu's place (limit:
-    ACT_CLAMPED_GATE's)."""
+    ACT_CLAMPED_GATE's, a number or the triple of _limits)."""
     _need(gu, "gu"); _need(out, "out", gu.dtype)
-    f = _fn("elementwise", "stratum_swiglu", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p])
-    _check(f(_ptr(gu), _ptr(out), dtype_code(gu.dtype), out.shape[0], out.shape[1], int(act), c_float(limit), _stream()),
-           "swiglu")
+    lim, first, beyond = _limits(limit)
+    f = _fn("elementwise", "stratum_swiglu",
+            [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_void_p])
+    _check(f(_ptr(gu), _ptr(out), dtype_code(gu.dtype), out.shape[0], out.shape[1], int(act), c_float(lim), first,
+             c_float(beyond), _stream()), "swiglu")
 
 
 def rope_store(qkv: torch.Tensor, token_pos: torch.Tensor, token_seq: torch.Tensor,
@@ -424,15 +432,17 @@ def _linear_shapes(x, w, bias, out, epilogue, what):
 
 
 def gemm_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
-                epilogue: int, act: int = ACT_NONE, limit: float = 0.0) -> None:
+                epilogue: int, act: int = ACT_NONE, limit=0.0) -> None:
     """bfloat16, at most 32 rows of x: the weight-streaming tensor-core kernel (see EPI_*; act as linear_simple's,
-    with EPI_SWIGLU the gate's; limit: ACT_CLAMPED_GATE's)."""
+    with EPI_SWIGLU the gate's; limit: ACT_CLAMPED_GATE's, as swiglu's)."""
+    lim, first, beyond = _limits(limit)
     M, N, Kd = _linear_shapes(x, w, bias, out, epilogue, "gemm_skinny")
     _need(x, "x", torch.bfloat16, contiguous=False)
     f = _fn("gemm_skinny", "stratum_gemm_skinny",
-            [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p])
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float,
+             c_void_p])
     _check(f(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), epilogue, M, N, Kd, x.stride(0), out.stride(0), act,
-             c_float(limit), _stream()), "gemm_skinny")
+             c_float(lim), first, c_float(beyond), _stream()), "gemm_skinny")
 
 
 _scratch_epoch = 0
@@ -495,7 +505,8 @@ class _EpiExtra(ctypes.Structure):
                 ("norm_parts", c_int), ("norm_ld", c_int), ("norm_size", c_float), ("norm_eps", c_float),
                 ("emit_ldx", c_int), ("emit_ld", c_int),
                 ("rope_pairs", c_int), ("bt_stride", c_int), ("n_q", c_int), ("n_kv", c_int), ("head_dim", c_int),
-                ("page_tokens", c_int), ("write_cache", c_int), ("act", c_int), ("act_limit", c_float)]
+                ("page_tokens", c_int), ("write_cache", c_int), ("act", c_int), ("act_limit", c_float),
+                ("limit_beyond", c_float), ("limit_first", c_int)]
 
 
 class GemmExtra:
@@ -508,15 +519,17 @@ class GemmExtra:
                   parts were written: `last_parts()` after the call);
     EPI_QKV_ROPE  the columns are query, key and value heads (pairs of rotated dimensions neighbours): queries
                   are rotated and stored to `out`, keys rotated and written, values written, into the paged cache;
-    activation    EPI_STORE applies ACT_* to what it stores, EPI_SWIGLU takes it for the gate's (limit: ACT_CLAMPED_GATE's).
+    activation    EPI_STORE applies ACT_* to what it stores, EPI_SWIGLU takes it for the gate's (limit: ACT_CLAMPED_GATE's,
+                  as swiglu's).
     """
 
     def __init__(self):
         self.c = _EpiExtra()
         self.keep = []                      # tensors whose memory the struct points into
 
-    def activation(self, act: int, limit: float = 0.0) -> "GemmExtra":
-        self.c.act, self.c.act_limit = int(act), float(limit)
+    def activation(self, act: int, limit=0.0) -> "GemmExtra":
+        self.c.act = int(act)
+        self.c.act_limit, self.c.limit_first, self.c.limit_beyond = _limits(limit)
         return self
 
     def scaled_rows(self, norm_ss: torch.Tensor, parts: int, size: int, eps: float) -> "GemmExtra":
@@ -685,7 +698,7 @@ class _GeneralAttention(ctypes.Structure):
                 ("token_pos", c_void_p), ("token_seq", c_void_p), ("block_table", c_void_p),
                 ("qb_seq", c_void_p), ("qb_tok0", c_void_p), ("qb_ntok", c_void_p),
                 ("part_o", c_void_p), ("part_ml", c_void_p), ("seq_start", c_void_p), ("sink", c_void_p),
-                ("head_scale", c_void_p), ("gate", c_void_p),
+                ("head_scale", c_void_p), ("slope", c_void_p), ("gate", c_void_p),
                 ("ldq", c_int), ("ldo", c_int), ("bt_stride", c_int), ("n_tokens", c_int),
                 ("n_heads", c_int), ("group", c_int), ("maps", c_int),
                 ("qk_dim", c_int), ("v_dim", c_int), ("n_k_heads", c_int), ("n_v_heads", c_int), ("v_in_k", c_int),
@@ -703,7 +716,8 @@ class AttentionShape:
     head (`group`), score maps per head, key and value sizes, whether the values are the first v_dim values of
     the key rows, scale, softcap (0: none), window (0: every key; keep_first: with a window, the positions below it stay
     visible), chunk (0: none; else a position sees only keys of its own chunk of that many positions, counted from
-    position 0), head_scale (float32 [n_heads] or None: a factor on the scores of each head), the query factor
+    position 0), head_scale (float32 [n_heads] or None: a factor on the scores of each head), slope (float32 [n_heads] or
+    None: slope * (distance from the key) is taken off the scores of each head), the query factor
     1 + temp_coef ln(floor((p + 1) / temp_every) + 1), and for two maps the combination
     (a_0 - lam a_1) / rms * out_scale with its eps and the column of the output gate (-1: none)."""
 
@@ -711,18 +725,18 @@ class AttentionShape:
                  softcap: float = 0.0, window: int = 0, temp_coef: float = 0.0, temp_every: int = 1,
                  lam: float = 0.0, out_scale: float = 1.0, eps: float = 0.0, gate_col: int = -1,
                  sink: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0,
-                 head_scale: Optional[torch.Tensor] = None):
+                 head_scale: Optional[torch.Tensor] = None, slope: Optional[torch.Tensor] = None):
         self.keep_first = int(keep_first) if window > 0 else 0
         self.n_heads, self.group, self.maps, self.qk_dim, self.v_dim = n_heads, group, maps, qk_dim, v_dim
         self.v_in_k, self.scale, self.softcap, self.window = bool(v_in_k), scale, softcap, window
         self.temp_coef, self.temp_every, self.lam, self.out_scale = temp_coef, temp_every, lam, out_scale
         self.eps, self.gate_col = eps, gate_col
-        for name, t in (("sink", sink), ("head_scale", head_scale)):
+        for name, t in (("sink", sink), ("head_scale", head_scale), ("slope", slope)):
             if t is not None:
                 _need(t, name, torch.float32)
                 if t.numel() != n_heads:
                     raise KernelError(f"attention: one {name} per head")
-        self.sink, self.head_scale, self.chunk = sink, head_scale, int(chunk)
+        self.sink, self.head_scale, self.slope, self.chunk = sink, head_scale, slope, int(chunk)
 
     @property
     def span(self) -> int:
@@ -738,6 +752,7 @@ class AttentionShape:
         p.lam, p.out_scale, p.eps, p.keep_first = self.lam, self.out_scale, self.eps, self.keep_first
         p.sink = None if self.sink is None else self.sink.data_ptr()
         p.head_scale = None if self.head_scale is None else self.head_scale.data_ptr()
+        p.slope = None if self.slope is None else self.slope.data_ptr()
         p.mask_chunk = self.chunk
 
 
@@ -973,6 +988,77 @@ def qk_norm_rope(proj: torch.Tensor, token_pos: torch.Tensor, token_seq: torch.T
     _check(f(ctypes.addressof(p), dtype_code(q_out.dtype), _stream()), "qk_norm_rope")
 
 
+# ------------------------------------------------------------------ queries, keys and values behind a short convolution
+class _ShortConv(ctypes.Structure):
+    """Mirror of struct ShortConv in csrc/short_conv.cu."""
+    _fields_ = [("proj", c_void_p), ("conv_w", c_void_p), ("lam", c_void_p), ("v_first_in", c_void_p),
+                ("v_first_out", c_void_p), ("q_out", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p),
+                ("state", c_void_p), ("token_pos", c_void_p), ("token_seq", c_void_p), ("block_table", c_void_p),
+                ("run_seq", c_void_p), ("run_row", c_void_p), ("run_n", c_void_p), ("seq_start", c_void_p),
+                ("seq_slot", c_void_p),
+                ("ld", c_int), ("ldq", c_int), ("ld_first", c_int), ("bt_stride", c_int), ("n_tokens", c_int),
+                ("n_runs", c_int), ("n_heads", c_int), ("n_kv", c_int), ("dim", c_int), ("v_dim", c_int),
+                ("page_tokens", c_int), ("write_cache", c_int), ("taps", c_int), ("state_stride", c_int)]
+
+
+def short_conv(proj: torch.Tensor, conv_w: Optional[torch.Tensor], step, runs, state: Optional[torch.Tensor],
+               block_table: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, n_heads: int,
+               n_kv: int, dim: int, v_dim: int, page_tokens: int, write_cache: bool, lam: Optional[torch.Tensor] = None,
+               v_first_in: Optional[torch.Tensor] = None, v_first_out: Optional[torch.Tensor] = None) -> None:
+    """Between a query/key/value projection (float32 [tokens, >= channels], channels = (n_heads + n_kv) * dim + n_kv *
+    v_dim) and attention: a causal convolution over time per channel (conv_w float32 [taps, channels], or None: none),
+    whose last taps - 1 inputs live in `state` (float32 [slots, >= (taps - 1) * channels]); values mixed with
+    v_first_in (lam float32 [1]: its share) or kept in v_first_out (both [tokens, >= n_kv * v_dim]); queries to q_out, keys
+    and values to the paged caches, all of one dtype.  step gives token_pos, token_seq, seq_start and seq_slot; runs: None
+    (one token per sequence) or (seq, first row, tokens) int32 tensors that cut every sequence's tokens from its first on
+    into runs of at least taps - 1 tokens (the last one of a sequence aside)."""
+    _need(proj, "proj", torch.float32, contiguous=False); _need(q_out, "q_out", contiguous=False)
+    for name in ("token_pos", "token_seq", "seq_start", "seq_slot"):
+        _need(getattr(step, name), name, torch.int32)
+    channels = (n_heads + n_kv) * dim + n_kv * v_dim
+    p = _ShortConv()
+    if conv_w is not None:
+        _need(conv_w, "conv_w", torch.float32)
+        p.taps = conv_w.shape[0]
+        if conv_w.dim() != 2 or conv_w.shape[1] != channels:
+            raise KernelError("short_conv: conv_w is [taps, channels]")
+        p.conv_w = conv_w.data_ptr()
+        if p.taps > 1:
+            _need(state, "state", torch.float32)
+            p.state, p.state_stride = state.data_ptr(), state.stride(0)
+    if proj.shape[1] < channels or proj.stride(1) != 1 or q_out.shape[0] != proj.shape[0] or q_out.shape[1] < n_heads * dim:
+        raise KernelError("short_conv: shapes disagree")
+    for name, t in (("v_first_in", v_first_in), ("v_first_out", v_first_out)):
+        if t is not None:
+            _need(t, name, q_out.dtype, contiguous=False)
+            if t.shape[0] != proj.shape[0] or t.shape[1] < n_kv * v_dim or (p.ld_first and p.ld_first != t.stride(0)):
+                raise KernelError(f"short_conv: {name} is [tokens, n_kv * v_dim]")
+            setattr(p, name, t.data_ptr())
+            p.ld_first = t.stride(0)
+    if v_first_in is not None:
+        _need(lam, "lam", torch.float32)
+        p.lam = lam.data_ptr()
+    p.proj, p.q_out, p.ld, p.ldq, p.n_tokens = proj.data_ptr(), q_out.data_ptr(), proj.stride(0), q_out.stride(0), proj.shape[0]
+    p.token_pos, p.token_seq = step.token_pos.data_ptr(), step.token_seq.data_ptr()
+    p.seq_start, p.seq_slot = step.seq_start.data_ptr(), step.seq_slot.data_ptr()
+    if runs is None:
+        p.n_runs = proj.shape[0]
+    else:
+        rs, rr, rn = runs
+        p.run_seq, p.run_row, p.run_n, p.n_runs = rs.data_ptr(), rr.data_ptr(), rn.data_ptr(), rs.numel()
+    p.n_heads, p.n_kv, p.dim, p.v_dim = n_heads, n_kv, dim, v_dim
+    p.page_tokens, p.write_cache = page_tokens, int(bool(write_cache))
+    if write_cache:
+        _need(block_table, "block_table", torch.int32, contiguous=False)
+        _need(k_cache, "k_cache", q_out.dtype); _need(v_cache, "v_cache", q_out.dtype)
+        if k_cache.shape[-1] != dim or v_cache.shape[-1] != v_dim:
+            raise KernelError("short_conv: the caches' rows and the head sizes disagree")
+        p.block_table, p.bt_stride = block_table.data_ptr(), block_table.stride(0)
+        p.k_cache, p.v_cache = k_cache.data_ptr(), v_cache.data_ptr()
+    f = _fn("short_conv", "stratum_short_conv", [c_void_p, c_int, c_void_p])
+    _check(f(ctypes.addressof(p), dtype_code(q_out.dtype), _stream()), "short_conv")
+
+
 # ------------------------------------------------------------------ the gated delta rule
 class _DeltaRule(ctypes.Structure):
     """Mirror of struct DeltaRule in csrc/delta_rule.cu."""
@@ -1081,7 +1167,7 @@ class _Gla(ctypes.Structure):
                 ("ld", c_int), ("ldo", c_int), ("n_tokens", c_int), ("n_seqs", c_int),
                 ("n_heads", c_int), ("dim", c_int), ("vdim", c_int), ("rank", c_int),
                 ("state_stride", c_int), ("write_state", c_int), ("ld_inner", c_int), ("rot_pairs", c_int),
-                ("eps", c_float), ("inv_tau", c_float), ("q_scale", c_float), ("reserved", c_float)]
+                ("eps", c_float), ("inv_tau", c_float), ("q_scale", c_float), ("silu_qkv", c_int), ("norm_all", c_int)]
 
 
 class GlaStep:
@@ -1094,10 +1180,11 @@ class GlaStep:
 
     With head_decay (float32 [heads]: a constant decay per head; rank 0) there is neither `cast` nor `decay`;
     `rotate(table, interleaved)` turns q and k in place by the step's (cos, sin) table float32 [tokens, pairs, 2], and
-    `recur` may take the tokens in chunks on tensor cores (`chunked`; see csrc/gla_chunked.cu) where `chunks_ok`."""
+    `recur` may take the tokens in chunks on tensor cores (`chunked`; see csrc/gla_chunked.cu) where `chunks_ok`.  silu_qkv:
+    `recur` takes q, k and v through silu; norm_all: `finish` norms all heads' read-outs together and gates by sigmoid."""
 
     def __init__(self, proj: torch.Tensor, n_heads: int, dim: int, vdim: int, rank: int, tau: float, q_scale: float,
-                 eps: float, head_decay: Optional[torch.Tensor] = None):
+                 eps: float, head_decay: Optional[torch.Tensor] = None, silu_qkv: bool = False, norm_all: bool = False):
         _need(proj, "proj", torch.float32, contiguous=False)
         p = self.p = _Gla()
         p.proj, p.ld, p.n_tokens = proj.data_ptr(), proj.stride(0), proj.shape[0]
@@ -1105,6 +1192,7 @@ class GlaStep:
         p.state_stride = n_heads * dim * vdim           # until recur() is told the real one
         p.ldo = n_heads * vdim
         p.eps, p.inv_tau, p.q_scale = float(eps), 1.0 / float(tau), float(q_scale)
+        p.silu_qkv, p.norm_all = int(bool(silu_qkv)), int(bool(norm_all))
         p.n_seqs = 1
         self.T, self.keep = proj.shape[0], [proj]
         if head_decay is not None:
@@ -1165,12 +1253,13 @@ class GlaStep:
         self._run(1, torch.float32, "gla_recur")
 
     def finish(self, gain: Optional[torch.Tensor], out: torch.Tensor) -> None:
-        """gain: float32 [vdim], or None: the norm has no weight."""
+        """gain: float32 [vdim] (norm_all: [heads * vdim]), or None: the norm has no weight."""
         _need(out, "out", contiguous=False)
         if gain is not None:
             _need(gain, "gain", torch.float32)
         p = self.p
-        if (gain is not None and gain.numel() != p.vdim) or out.shape[0] != self.T or out.shape[1] < p.n_heads * p.vdim or not p.o_raw:
+        n_gain = p.vdim * (p.n_heads if p.norm_all else 1)
+        if (gain is not None and gain.numel() != n_gain) or out.shape[0] != self.T or out.shape[1] < p.n_heads * p.vdim or not p.o_raw:
             raise KernelError("gla: shapes disagree, or the recurrence has not run")
         p.gain = None if gain is None else gain.data_ptr()
         p.out, p.ldo = out.data_ptr(), out.stride(0)
@@ -1317,20 +1406,21 @@ class _MoeRoute(ctypes.Structure):
                 ("chosen", c_void_p), ("weights", c_void_p),
                 ("ldx", c_int), ("ldd", c_int), ("n_tokens", c_int), ("width", c_int),
                 ("n_experts", c_int), ("top", c_int), ("n_groups", c_int), ("keep", c_int),
-                ("scale", c_float), ("reserved", c_float), ("w_gate", c_void_p), ("score", c_int), ("renorm", c_int),
+                ("scale", c_float), ("group_score", c_int), ("w_gate", c_void_p), ("score", c_int), ("renorm", c_int),
                 ("bias", c_void_p)]
 
 
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], dense: torch.Tensor,
               chosen: torch.Tensor, weights: torch.Tensor, top: int, n_groups: int, keep: int, scale: float,
               softmax: bool = False, renorm: bool = True, w_gate: Optional[torch.Tensor] = None,
-              bias: Optional[torch.Tensor] = None) -> None:
+              bias: Optional[torch.Tensor] = None, group_max: bool = False) -> None:
     """Routing with a choice correction and groups (see csrc/moe_router.cu): scores by sigmoid, or by softmax over all
     experts; the chosen scores divided by their sum (renorm) or left as they are.  x [tokens, width] float32 or
     bfloat16; w_router float32 [experts, width]; correction float32 [experts] or None; dense float32 [tokens, >=
     experts] (weights, zeros for experts not chosen); chosen int32 and weights float32 [tokens, top].  w_gate
     float32 [width]: dense[:, experts] receives sigmoid(x . w_gate), the gate of a shared expert.  bias float32
-    [experts]: added to the router's products before they are scored."""
+    [experts]: added to the router's products before they are scored.  group_max: a group's score is its largest choice
+    score, not the sum of its two largest."""
     _need(x, "x", contiguous=False); _need(w_router, "w_router", torch.float32)
     _need(dense, "dense", torch.float32, contiguous=False)
     _need(chosen, "chosen", torch.int32); _need(weights, "weights", torch.float32)
@@ -1342,7 +1432,7 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, correction: Optional[torc
         raise KernelError("moe_route: shapes disagree")
     p = _MoeRoute()
     p.x, p.w_router, p.correction = x.data_ptr(), w_router.data_ptr(), (0 if correction is None else correction.data_ptr())
-    p.score, p.renorm = int(bool(softmax)), int(bool(renorm))
+    p.score, p.renorm, p.group_score = int(bool(softmax)), int(bool(renorm)), int(bool(group_max))
     if bias is not None:
         _need(bias, "bias", torch.float32)
         if bias.numel() != E:
@@ -1468,12 +1558,17 @@ def attention_tile(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
 def attention_tc(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, token_pos: torch.Tensor,
                  block_table: torch.Tensor, qblocks, out: torch.Tensor, n_q: int, n_kv: int, head_dim: int,
                  page_tokens: int, window: int, scale: float, halves: int = 1, split: bool = False, chunk: int = 0,
-                 gate: Optional[torch.Tensor] = None) -> None:
+                 gate: Optional[torch.Tensor] = None, slope: Optional[torch.Tensor] = None) -> None:
     """bfloat16 attention for prompts on tcgen05/TMEM: query tiles of halves * 128 / (n_q / n_kv) tokens (qblocks
     as for attention_tile).  halves 2: a CTA owns 256 query rows whose two halves share every key and value tile.
     head_dim 64 or 128, group size dividing 128, pages of 64 tokens.  split (with halves 2): the probabilities keep 16
     bits of mantissa (two bfloat16 parts) instead of 8; chunk: a position sees only keys of its own chunk of that many
-    positions (0: all); gate (float32 [tokens, n_q * head_dim]): the output times sigmoid(gate), element by element."""
+    positions (0: all); gate (float32 [tokens, n_q * head_dim]): the output times sigmoid(gate), element by element; slope
+    (float32 [n_q], with split): slope * (distance from the key) is taken off the scores."""
+    if slope is not None:
+        _need(slope, "slope", torch.float32)
+        if slope.numel() != n_q:
+            raise KernelError("attention_tc: one slope per query head")
     if gate is not None:
         _need(gate, "gate", torch.float32, contiguous=False)
         if gate.shape[0] != qkv.shape[0] or gate.shape[1] < n_q * head_dim or gate.stride(1) != 1:
@@ -1485,12 +1580,12 @@ def attention_tc(qkv: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor
     f = _fn("attention_tc", "stratum_attention_tc",
             [c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
              c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int,
-             c_void_p, c_int, c_void_p, c_void_p])
+             c_void_p, c_int, c_void_p, c_void_p, c_void_p])
     _check(f(_ptr(qkv), qkv.stride(0), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0], _ptr(token_pos),
              _ptr(block_table), block_table.stride(0), _ptr(qs), _ptr(qt), _ptr(qn), qs.numel(), _ptr(out),
              out.stride(0), qkv.shape[0], n_q, n_kv, head_dim, page_tokens, window, c_float(scale), halves,
-             int(bool(split)), int(chunk), _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(status_word()),
-             _stream()), "attention_tc")
+             int(bool(split)), int(chunk), _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(slope),
+             _ptr(status_word()), _stream()), "attention_tc")
 
 
 _stream_scratch = None

@@ -1,4 +1,4 @@
-from . import (attention, block, delta_rule, differential_attention, embedding, latent_attention, linear_attention,  # noqa: F401
+from . import (attention, block, conv_attention, delta_rule, differential_attention, embedding, latent_attention, linear_attention,  # noqa: F401
                linear_recurrence, mixer_mean, mlp, moe, norm, reentry, retention, rope, sink_attention, state_space)  # noqa: F401  (registers the built-in parts)
 from .base import (Arrangement, Embedding, FeedForward, Head, Mixer, Norm, Part, PositionEncoding,
                    RotaryTable, Runtime)

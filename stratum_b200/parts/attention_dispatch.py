@@ -128,7 +128,7 @@ def _plain_heads(shape, q: torch.Tensor, cache, out: torch.Tensor, gate) -> bool
 def run_general(att, shape, q: torch.Tensor, cache, step, out: torch.Tensor, gate=None) -> None:
     """Attention of the shapes kernels.AttentionShape describes (key and value sizes of their own, values inside the
     key rows, several maps per head): q [tokens, *] holds head j's map m at column (j * maps + m) * qk_dim.
-    bfloat16 prompts of heads that need nothing beyond chunks, a window and a gate: the tcgen05 kernel, with
+    bfloat16 prompts of heads that need nothing beyond chunks, a window, a distance bias and a gate: the tcgen05 kernel, with
     probabilities of 16 bits; bfloat16 with sizes in multiples of 8: the tensor-core kernel (decode steps: the keys cut into ranges that
     fill the GPU; prompts: query blocks of 16 rows); everything else: the CUDA-core kernel, float32 throughout.
     gate (float32 [tokens, heads * v_dim] or None): pre-activations of an output gate per element.
@@ -138,7 +138,7 @@ def run_general(att, shape, q: torch.Tensor, cache, step, out: torch.Tensor, gat
             and os.environ.get("STRATUM_GENERAL_ATTENTION_TC", "1") != "0":
         K.attention_tc(q, cache.k, cache.v, step.token_pos, cache.block_table, step.query_blocks(2 * (128 // shape.group)),
                        out, shape.n_heads, shape.n_heads // shape.group, shape.qk_dim, PAGE_TOKENS, shape.window, shape.scale,
-                       halves=2, split=True, chunk=shape.chunk, gate=gate)
+                       halves=2, split=True, chunk=shape.chunk, gate=gate, slope=shape.slope)
         return
     if (not K.attention_general_mma_ok(shape, q, out, PAGE_TOKENS, gate)
             or os.environ.get("STRATUM_GENERAL_ATTENTION_MMA", "1") == "0"):

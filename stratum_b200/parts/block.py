@@ -51,7 +51,8 @@ class ParallelResidual(Arrangement):
     """x += mixer(norm_a(x)) + feed_forward(norm_b(x)): both sublayers read the same x, each through a norm of its own,
     and both add into the stream.  Both norms run before either sublayer writes; where they are RMS norms of one size
     and eps (which is what the library's models give) one kernel reads the row once, takes one sum of squares and
-    writes both outputs.  A layer may have no feed-forward."""
+    writes both outputs.  A layer may have one norm for both sublayers (no `feed_forward_norm`): both then read its rows.
+    A layer may have no feed-forward."""
     replays_prompts = True
     slots = {"mixer_norm": "norm", "mixer": "mixer", "feed_forward_norm": "norm", "feed_forward": "feed_forward"}
     optional = ("feed_forward_norm", "feed_forward")
@@ -60,7 +61,10 @@ class ParallelResidual(Arrangement):
         norm_a, mixer = layer.part("mixer_norm"), layer.part("mixer")
         norm_b, ff = layer.part("feed_forward_norm"), layer.part("feed_forward")
         if ff is None or norm_b is None:
-            mixer.forward(norm_a.forward(x), x, step, cache)
+            xn = norm_a.forward(x)
+            mixer.forward(xn, x, step, cache)
+            if ff is not None:
+                ff.forward(xn, x, step)
             return
         pair = getattr(norm_a, "forward_pair", None)
         both = pair(x, norm_b) if pair is not None else None

@@ -65,7 +65,7 @@ def takes_tensor_cores(x: torch.Tensor, w: torch.Tensor, extras: bool) -> bool:
 
 
 def run(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, mode: int,
-        extra=None, act: int = 0, limit: float = 0.0) -> None:
+        extra=None, act: int = 0, limit=0.0) -> None:
     """out (=|+=) epilogue(x @ w.T + bias); see the EPI_* modes in kernels.py.  act: with STORE an activation
     applied to what is stored, with SWIGLU the gate's activation in silu's place (kernels.ACT_*; limit: the clamped
     gate's), by whichever kernel takes the call."""

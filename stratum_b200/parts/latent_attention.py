@@ -24,7 +24,9 @@ Two optional pieces, each a parameter.  Queries through a latent of their own (`
 q = Wuq cq; the down projection joins the fused first product, the norm runs in place on its stretch of the row
 (float32 statistic), and the up projection writes the queries where the direct projection would have.  A gate per
 head (`gate`): head j's output times sigmoid(Wg h)_j, whose pre-activation is one more column stretch of the first
-product; the sigmoid is taken in float32 on the heads' outputs, in front of the output projection.
+product; the sigmoid is taken in float32 on the heads' outputs, in front of the output projection.  Without a position
+encoding there is no rotated part (`rot_dim` 0): the cache keeps c alone.  A sink (`sink`): a learned number per head
+whose exponential joins the softmax's denominator.
 """
 from __future__ import annotations
 
@@ -56,15 +58,15 @@ def padded(n: int, to: int = 8) -> int:
 class LatentAttention(Mixer):
     """params: hidden, n_heads, head_dim (the unrotated query/key size), rot_dim, v_dim, kv_rank, scale, eps (of
     the latents' norms), position (PartSpec of a rotating position encoding over at most rot_dim dimensions, pairs
-    (i, i + n/2) or neighbours (2i, 2i + 1) as the encoding says), window (0 = all keys), q_rank (None or 0: queries
+    (i, i + n/2) or neighbours (2i, 2i + 1) as the encoding says; None: nothing is rotated, rot_dim may be 0), sink, window (0 = all keys), q_rank (None or 0: queries
     projected directly from the input; else the size of the queries' latent), gate (a sigmoid gate per head on the
     heads' outputs), prefix, and the tensor names q, dkv, dkv_norm, uk, uv, o, and with q_rank dq, dq_norm, uq, with
-    gate g (defaults: those words, with "dkv.norm" and "dq.norm")."""
+    gate g, with sink sink_tensor (defaults: those words, with "dkv.norm", "dq.norm" and "sink")."""
     stores_output = True
 
     @property
     def replays_prompts(self) -> bool:
-        return bool(getattr(self.position, "replays_prompts", False))
+        return self.position is None or bool(getattr(self.position, "replays_prompts", False))
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
@@ -73,16 +75,20 @@ class LatentAttention(Mixer):
                                               int(spec["kv_rank"]))
         self.scale, self.eps = float(spec["scale"]), float(spec["eps"])
         self.window = int(spec.get("window", 0) or 0)
-        pos: PartSpec = spec["position"]
-        self.position = find_part("position", pos.kind)(pos, runtime)
-        layout = self.position.pair_layout()
-        if layout is None or 2 * layout[0] > self.r:
-            raise ValueError("latent attention rotates pairs of at most rot_dim dimensions")
-        self.interleaved = bool(layout[1])
+        pos: Optional[PartSpec] = spec.get("position")
+        self.position = find_part("position", pos.kind)(pos, runtime) if pos is not None else None
+        self.interleaved = False
+        if self.position is not None:
+            layout = self.position.pair_layout()
+            if layout is None or 2 * layout[0] > self.r:
+                raise ValueError("latent attention rotates pairs of at most rot_dim dimensions")
+            self.interleaved = bool(layout[1])
+        self.has_sink = bool(spec.get("sink", False))
         self.q_rank = int(spec.get("q_rank") or 0)
         self.gate = bool(spec.get("gate", False))
         self.names = {k: self.prefix + str(spec.get(k, k.replace("_norm", ".norm")))
                       for k in ("q", "dkv", "dkv_norm", "uk", "uv", "o", "dq", "dq_norm", "uq", "g")}
+        self.names["sink"] = self.prefix + str(spec.get("sink_tensor", "sink"))
         # columns of a token's row of projections: [queries | c' kr | the queries' latent | the gates], every
         # stretch starting at a multiple of 8 (16 bytes in bfloat16: rows a product may read or write by vectors)
         self.q_cols = self.n_heads * (self.d + self.r)
@@ -91,8 +97,7 @@ class LatentAttention(Mixer):
         self.g_col = self.cq_col + padded(self.q_rank)
         self.width = (self.g_col + self.n_heads if self.gate else
                       self.cq_col + self.q_rank if self.q_rank else self.kv_col + self.rank + self.r)
-        self.shape = K.AttentionShape(self.n_heads, self.n_heads, 1, self.rank + self.r, self.rank, True, self.scale,
-                                      window=self.window)
+        self.shape: Optional[K.AttentionShape] = None
         self.w_in: Optional[Linear] = None
         self.w_uq: Optional[Linear] = None
         self.w_o: Optional[Linear] = None
@@ -115,6 +120,8 @@ class LatentAttention(Mixer):
             t[n["q"]] = TensorSpec((self.q_cols, self.hidden))
         if self.gate:
             t[n["g"]] = TensorSpec((H, self.hidden))
+        if self.has_sink:
+            t[n["sink"]] = TensorSpec((H,), role="vector", init="zeros")
         return t
 
     def _stack_rows(self, pieces) -> torch.Tensor:
@@ -141,6 +148,9 @@ class LatentAttention(Mixer):
             pieces.append((self.g_col, weights[n["g"]]))
         self.w_in = Linear(self.runtime, self._stack_rows(pieces))
         self.gain = weights[n["dkv_norm"]]
+        self.inv_freq = None if self.position is None else self.position.rotary().inv_freq
+        sink = weights[n["sink"]].contiguous() if self.has_sink else None
+        self.shape = K.AttentionShape(H, H, 1, self.rank + self.r, self.rank, True, self.scale, window=self.window, sink=sink)
         # head j carries its plain query into the latent space with Wuk_j^T: a matrix [rank, d] per head
         self.uk = HeadLinear(self.runtime, weights[n["uk"]].view(H, self.d, self.rank).transpose(1, 2).contiguous())
         self.uv = HeadLinear(self.runtime, weights[n["uv"]].view(H, self.dv, self.rank))
@@ -154,7 +164,7 @@ class LatentAttention(Mixer):
             stack[:, d:, rank:] = torch.eye(r, dtype=torch.bfloat16, device=stack.device)
             self.w_keys = Linear(self.runtime, stack.view(H * (d + r), rank + r))
             self.w_values = Linear(self.runtime, weights[n["uv"]])
-            self.head_shape = K.AttentionShape(H, 1, 1, d + r, self.dv, False, self.scale, window=self.window)
+            self.head_shape = K.AttentionShape(H, 1, 1, d + r, self.dv, False, self.scale, window=self.window, sink=sink)
 
     def cache_spec(self) -> KVSpec:
         return KVSpec(1, self.rank + self.r, self.window, f"latent_{self.rank}_then_rotated", value_heads=0)
@@ -165,7 +175,7 @@ class LatentAttention(Mixer):
         sequences begin) in which every sequence begins at position 0 and the longest brings PER_HEAD_MIN_TOKENS."""
         if self.w_keys is None or step.all_single or step.fixed_qblocks is not None or step.sizes_seen is not None:
             return False
-        if not cache.writes or self.window or os.environ.get("STRATUM_LATENT_PER_HEAD", "1") == "0":
+        if not cache.writes or os.environ.get("STRATUM_LATENT_PER_HEAD", "1") == "0":
             return False
         before = (step.host or {}).get("before")
         return bool(before) and all(b == 0 for b in before) and step.max_new >= PER_HEAD_MIN_TOKENS
@@ -183,7 +193,7 @@ class LatentAttention(Mixer):
         rows = self.runtime.empty(T, padded(rank + r))            # [c | kr] of the step's tokens
         K.mixer_prep(proj, step.token_pos, step.token_seq, cache.block_table, cache.k, None, PAGE_TOKENS, True,
                      queries=(H, d + r, 0), q_rot_off=d, keys=(1, rank + r, self.kv_col), k_rot_off=rank,
-                     inv_freq=self.position.rotary().inv_freq, k_norm_gain=self.gain, eps=self.eps, k_out=rows,
+                     inv_freq=self.inv_freq, k_norm_gain=self.gain, eps=self.eps, k_out=rows,
                      interleaved=self.interleaved)
         # 64 rows beyond the step's: the last tile of the last sequence reads (and ignores) them
         keys = self.runtime.empty(T + PAGE_TOKENS, padded(H * (d + r)))
@@ -215,7 +225,7 @@ class LatentAttention(Mixer):
         q_lat = self.runtime.empty(T, padded(H * (rank + r)))
         K.mixer_prep(proj, step.token_pos, step.token_seq, cache.block_table, cache.k, None, PAGE_TOKENS, cache.writes,
                      queries=(H, d + r, 0), q_rot_off=d, keys=(1, rank + r, self.kv_col), k_rot_off=rank,
-                     inv_freq=self.position.rotary().inv_freq, k_norm_gain=self.gain, eps=self.eps,
+                     inv_freq=self.inv_freq, k_norm_gain=self.gain, eps=self.eps,
                      q_out=q_lat, q_out_step=rank + r, q_out_off=rank, interleaved=self.interleaved)
         self.uk(proj, d + r, q_lat, rank + r)
         mixed = self.runtime.empty(T, padded(H * rank))

@@ -28,14 +28,14 @@ class Linear:
         self.out_features, self.in_features = weight.shape
 
     def __call__(self, x, out: Optional[torch.Tensor] = None, mode: int = STORE, emit=None, extra=None,
-                 act: int = 0, limit: float = 0.0) -> torch.Tensor:
+                 act: int = 0, limit=0.0) -> torch.Tensor:
         """mode STORE: new tensor of x's dtype; ADD_TO_F32: out (float32) += y; STORE_F32: float32 out;
         SWIGLU: rows of W alternate gate and up, out[m][j] = silu(y[m][2j]) * y[m][2j+1] in x's dtype;
         QKV_ROPE: see kernels.GemmExtra (extra carries the cache and the rotation table; out: the query rows).
         x may be NormedRows (the product then applies the norm's row factors).  emit: a Handover that the
         ADD_TO_F32 product honours where it can (emit.result is then set).  act: with STORE an activation the
         product applies to what it stores, with SWIGLU the gate's activation in silu's place (kernels.ACT_*; limit: the
-        clamped gate's)."""
+        clamped gate's, a number or (limit, first, beyond): `beyond` from output column `first` on)."""
         from . import gemm_dispatch
         from .base import NormedRows
         normed = x if isinstance(x, NormedRows) else None

@@ -29,7 +29,10 @@ matrix, Wdown act(Wup h), with the activation named (`gated` false, `activation`
 multiplied by sigmoid(w_sg . h), one number per token (`shared_gate`: the name of that row of weights): the router's
 kernel takes that dot product with the experts' and leaves the gate beside the experts' weights; and a bias on the
 router's logits (`router_bias`: tensor router.b).  Softmax scores over all experts, renormalised over the chosen ones,
-are the softmax over the chosen logits alone: a design that states its weights that way sets `score: softmax`.
+are the softmax over the chosen logits alone: a design that states its weights that way sets `score: softmax`.  A group's
+score may be its largest choice score (`group_score: max`), and experts may have the clamped gate of parts/mlp.py, the
+routed ones with one limit and the shared one with its own (`activation: clamped`, `limit`, `shared_limit`): in the
+stacked product the shared expert's columns come last, so its limit holds from a column on.
 """
 from __future__ import annotations
 
@@ -42,7 +45,7 @@ import torch
 from .. import kernels as K
 from .base import FeedForward
 from .linear import ADD_TO_F32, STORE, STORE_F32, SWIGLU, Linear
-from .mlp import GATE_ACTS, interleave_rows
+from .mlp import CLAMPED, GATE_ACTS, interleave_rows
 from .registry import register_part
 from .spec import TensorSpec
 
@@ -57,7 +60,8 @@ GROUPED_MIN_ROWS = int(os.environ.get("STRATUM_MOE_GROUPED_MIN_ROWS", 96))
 class RoutedExperts(FeedForward):
     """params: hidden, n_experts, top, scale, n_groups, keep, intermediate (of an expert), shared_intermediate (of
     the shared expert; None: none), prefix; score ("sigmoid" or "softmax"), renorm, correction, gated, activation
-    ("silu", "gelu_tanh", "gelu_erf", "relu_sq"), shared_gate (tensor name under the prefix, or None), router_bias.
+    ("silu", "gelu_tanh", "gelu_erf", "relu_sq", "clamped" with limit and shared_limit), shared_gate (tensor name under the
+    prefix, or None), router_bias, group_score ("top2" or "max").
     Tensors: router, router.b, correction, e<i>.gate / .up / .down, shared.gate / .up / .down (no .gate when not gated)."""
     stores_output = True
 
@@ -80,10 +84,18 @@ class RoutedExperts(FeedForward):
         self.has_correction = bool(spec.get("correction", True))
         self.gated = bool(spec.get("gated", True))
         act = spec.get("activation", "silu")
-        if act not in GATE_ACTS or (not self.gated and act == "silu"):
+        if (act not in GATE_ACTS and act != CLAMPED) or (not self.gated and act in ("silu", CLAMPED)):
             raise ValueError(f"routed_experts: activation {act!r} is not known"
                              + ("" if self.gated else " to experts without a gate"))
-        self.act = GATE_ACTS[act]
+        self.act = K.ACT_CLAMPED_GATE if act == CLAMPED else GATE_ACTS[act]
+        self.limit = self.shared_limit = 0.0
+        if act == CLAMPED:
+            self.limit = float(spec["limit"])
+            self.shared_limit = float(spec["shared_limit"]) if self.shared_ff else self.limit
+        group_score = spec.get("group_score", "top2")
+        if group_score not in ("top2", "max"):
+            raise ValueError(f"routed_experts: group_score {group_score!r} is neither 'top2' nor 'max'")
+        self.group_max = group_score == "max"
         self.shared_gate = spec.get("shared_gate") if self.shared_ff else None
         self.has_router_bias = bool(spec.get("router_bias", False))
         self.correction = self.w_gate = self.router_bias = None
@@ -140,13 +152,14 @@ class RoutedExperts(FeedForward):
         chosen = self.runtime.empty(T, self.top, dtype=torch.int32)
         weights = self.runtime.empty(T, self.top, dtype=torch.float32)
         K.moe_route(xin, self.router, self.correction, dense, chosen, weights, self.top, self.n_groups, self.keep,
-                    self.scale, softmax=self.softmax, renorm=self.renorm, w_gate=self.w_gate, bias=self.router_bias)
+                    self.scale, softmax=self.softmax, renorm=self.renorm, w_gate=self.w_gate, bias=self.router_bias,
+                    group_max=self.group_max)
         return dense, chosen, weights
 
-    def _first(self, lin: Linear, x: torch.Tensor) -> torch.Tensor:
+    def _first(self, lin: Linear, x: torch.Tensor, limit) -> torch.Tensor:
         """An expert's (or all experts') activations: act(gate) * up, or act(up) where the experts have no gate."""
         if self.gated:
-            return lin(x, mode=SWIGLU, act=self.act)
+            return lin(x, mode=SWIGLU, act=self.act, limit=limit)
         return lin(x, mode=STORE, act=self.act)
 
     def grouped(self, step, n_tokens: int) -> bool:
@@ -173,7 +186,7 @@ class RoutedExperts(FeedForward):
         T = xin.shape[0]
         E = self.n_experts
         if not self.grouped(step, T):
-            a = self._first(self.gate_up, xin)
+            a = self._first(self.gate_up, xin, (self.limit, E * self.ff, self.shared_limit))
             K.scale_column_blocks(a, dense, self.ff, E)
             if self.w_gate is not None:                   # the shared expert's stretch times the token's gate
                 K.scale_column_blocks(a[:, E * self.ff:], dense[:, E:], self.shared_ff, 1)
@@ -187,11 +200,11 @@ class RoutedExperts(FeedForward):
         at = 0
         for e, n in enumerate(counts):
             if n:
-                a = self._first(self.gate_up_of[e], rows[at:at + n])
+                a = self._first(self.gate_up_of[e], rows[at:at + n], self.limit)
                 self.down_of[e](a, out=outs[at:at + n], mode=STORE_F32)
                 at += n
         if self.shared_ff:
-            a = self._first(self.gate_up_of[E], xin)
+            a = self._first(self.gate_up_of[E], xin, self.shared_limit)
             if self.w_gate is not None:
                 K.scale_column_blocks(a, dense[:, E:], self.shared_ff, 1)
             self.down_of[E](a, out=residual, mode=STORE_F32 if store else ADD_TO_F32)
