@@ -8,6 +8,7 @@
     python bench.py --compare vitinex       # the Vitinex decoder beside the Dabodra and the Llama decoder of equal size
     python bench.py --compare mokatar       # the Mokatar decoder beside the same two
     python bench.py --compare getizen       # the Getizen decoder beside the Mokatar and the Llama decoder of equal size
+    python bench.py --compare memipel       # the Memipel decoder beside the Getizen, Vitinex and Llama decoders
 
 Prints ONE JSON line.  `value` is decoded tokens per second at the given batch, with every
 sequence's cache filled to the given context at the end of the timed steps (so the timed steps
@@ -208,6 +209,37 @@ def getizen_config(size, n_layers):
                                     "norm": {"eps": 1e-5, "groups": 2}, "postln_alpha": 1.5, "layers": layers})
 
 
+# --compare memipel: the same widths, heads and vocabulary, beside the Getizen decoder (the closest one here in attention
+# that is cut off behind 1,024 positions, linear attention with the same state of 128 x 128 per head and clamped gates),
+# the Vitinex decoder (the closest one in latent attention with a query latent and in routed experts by softmax) and the
+# Llama decoder.  Of every four layers two are attention behind short convolutions, one is latent attention, one is
+# lightning attention; the first layer's feed-forward is dense (2 x ff = 3 x llama_inner), the others have eight routed
+# experts of which a token uses two, and a shared expert, sized so that a token's active weights equal the Llama decoder's.
+MEMIPEL_SIZES = {
+    "1b": {"dim": 128, "vdim": 128, "window": 1024, "latent": {"dim": 64, "vdim": 64, "kv_rank": 256, "q_rank": 768},
+           "light_dim": 128, "light_vdim": 128, "experts": 8, "top": 2, "ff": 1408, "shared": 2688},
+    "8b": {"dim": 128, "vdim": 128, "window": 1024, "latent": {"dim": 128, "vdim": 128, "kv_rank": 512, "q_rank": 1536},
+           "light_dim": 128, "light_vdim": 128, "experts": 8, "top": 2, "ff": 2816, "shared": 5248},
+}
+
+
+def memipel_config(size, n_layers):
+    from stratum_b200.config import MemipelConfig
+    z, m = COMPARE_SIZES[size], MEMIPEL_SIZES[size]
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": m["dim"], "vdim": m["vdim"], "scale": m["dim"] ** -0.5,
+           "conv": 4, "v_mix": True, "mask": {"size": m["window"]}}
+    lat = dict(m["latent"], heads=z["heads"], scale=m["latent"]["dim"] ** -0.5, mask={"size": m["window"]})
+    light = {"heads": z["heads"], "dim": m["light_dim"], "vdim": m["light_vdim"],
+             "decay": [1.0 - 2.0 ** (-5 - 5 * h / z["heads"]) for h in range(z["heads"])]}
+    moe = {"kind": "moe", "router": {"experts": m["experts"], "top": m["top"], "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": m["ff"], "limit": 7.0}, "shared": {"ff": m["shared"], "limit": 9.0}}
+    kinds = [("attention", att), ("attention", att), ("lightning", light), ("latent_attention", lat)]
+    layers = [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1],
+               "mlp": moe if i else {"kind": "dense", "ff": 3 * z["llama_inner"] // 2}} for i in range(n_layers)]
+    return MemipelConfig.from_dict({"architecture": "Memipel", "vocab": z["vocab"], "width": z["width"],
+                                    "norm": {"eps": 1e-5}, "layers": layers})
+
+
 def llama_like(size, n_layers):
     from stratum_b200.config import LlamaConfig
     z = COMPARE_SIZES[size]
@@ -247,8 +279,9 @@ def kernel_times(llm, batch, context, prefill_tokens, vocab, rng):
 
 
 def compare_models(args, rng):
-    """Prefill and decode throughput of the Nibelorn, the Dabodra, the Vitinex, the Mokatar or the Getizen decoder beside
-    a Llama decoder of equal size (Vitinex and Mokatar also beside the Dabodra, Getizen beside the Mokatar decoder): one
+    """Prefill and decode throughput of the Nibelorn, the Dabodra, the Vitinex, the Mokatar, the Getizen or the Memipel
+    decoder beside a Llama decoder of equal size (Vitinex and Mokatar also beside the Dabodra, Getizen beside the Mokatar,
+    Memipel beside the Getizen and the Vitinex decoder): one
     prompt of --prefill-tokens, and decode steps of --batch sequences at --context tokens (random bf16 weights,
     device-timed as the main workload is); with --kernels also the device time of every kernel of one prompt and one
     decode step.  One JSON line."""
@@ -257,9 +290,10 @@ def compare_models(args, rng):
     n_layers = args.layers or 8
     which = args.compare
     make = {"nibelorn": nibelorn_config, "dabodra": dabodra_config, "vitinex": vitinex_config,
-            "mokatar": mokatar_config, "getizen": getizen_config}[which]
+            "mokatar": mokatar_config, "getizen": getizen_config, "memipel": memipel_config}[which]
     others = [("llama", llama_like)] + ([("dabodra", dabodra_config)] if which in ("vitinex", "mokatar") else []) \
-        + ([("mokatar", mokatar_config)] if which == "getizen" else [])
+        + ([("mokatar", mokatar_config)] if which == "getizen" else []) \
+        + ([("getizen", getizen_config), ("vitinex", vitinex_config)] if which == "memipel" else [])
     out = {"compare": which, "layers": n_layers, "batch": args.batch, "context": args.context,
            "prefill_tokens": args.prefill_tokens, "dtype": "bf16", "data": "synthetic: random-init weights",
            "sizes": {}}
@@ -517,10 +551,11 @@ def main() -> int:
                     help="prompt length of --prefill-only (the default JSON line always uses 2,048)")
     ap.add_argument("--shape", default="llama3.1-8b", choices=["llama3.1-8b"] + sorted(OTHER_SHAPES),
                     help="layer sizes for the short lines of --decode-only / --prefill-only")
-    ap.add_argument("--compare", default=None, choices=["nibelorn", "dabodra", "vitinex", "mokatar", "getizen"],
+    ap.add_argument("--compare", default=None, choices=["nibelorn", "dabodra", "vitinex", "mokatar", "getizen", "memipel"],
                     help="instead of the main workload: prefill and decode throughput of the Nibelorn, the Dabodra, "
-                         "the Vitinex, the Mokatar or the Getizen decoder beside a Llama decoder of equal size (Vitinex "
-                         "and Mokatar also beside Dabodra, Getizen beside Mokatar), at 1B-like and 8B-like layer sizes "
+                         "the Vitinex, the Mokatar, the Getizen or the Memipel decoder beside a Llama decoder of equal "
+                         "size (Vitinex and Mokatar also beside Dabodra, Getizen beside Mokatar, Memipel beside Getizen "
+                         "and Vitinex), at 1B-like and 8B-like layer sizes "
                          "(--layers of them, default 8)")
     ap.add_argument("--kernels", action="store_true",
                     help="with --compare: also the device time of every kernel of one prompt and one decode step")
