@@ -165,10 +165,28 @@ def route(z, top, count=1, keep=1):
     return out
 
 
-def experts(f, W, h, pre):
+def route_margin(z, top, count=1, keep=1):
+    """How far (in logits) the nearest of all choices of groups and of experts is from turning out otherwise."""
+    T, E = z.shape
+    best = z.reshape(T, count, E // count).max(axis=-1)
+    near = np.inf
+    for t in range(T):
+        order = np.argsort(-best[t], kind="stable")
+        if keep < count:
+            near = min(near, best[t, order[keep - 1]] - best[t, order[keep]])
+        can = np.sort([z[t, e] for e in range(E) if e // (E // count) in order[:keep]])[::-1]
+        if top < len(can):
+            near = min(near, can[top - 1] - can[top])
+    return near
+
+
+def experts(f, W, h, pre, margins=None):
     r = f["router"]
     gr = r.get("groups") or {"count": 1, "keep": 1}
-    weights = route(linear(h, W[pre + "router"]), r["top"], gr["count"], gr["keep"])
+    z = linear(h, W[pre + "router"])
+    if margins is not None:
+        margins.append(route_margin(z, r["top"], gr["count"], gr["keep"]))
+    weights = route(z, r["top"], gr["count"], gr["keep"])
     y = np.zeros_like(np.asarray(h, F64))
     for e in range(r["experts"]):
         y += weights[:, e:e + 1] * clamped_expert(W, h, f"{pre}e{e}.", f["expert"]["limit"])
@@ -177,13 +195,13 @@ def experts(f, W, h, pre):
     return y
 
 
-def feed_forward(f, W, h, pre):
-    return dense(W, h, pre) if f["kind"] == "dense" else experts(f, W, h, pre)
+def feed_forward(f, W, h, pre, margins=None):
+    return dense(W, h, pre) if f["kind"] == "dense" else experts(f, W, h, pre, margins)
 
 
-def forward(cfg, W, tokens, residuals=None, noise=None):
-    """Logits [T, vocab]; residuals: a list that receives the stream after every layer; noise: called on every norm's
-    output (a test that asks how far rounding of a given width reaches)."""
+def forward(cfg, W, tokens, residuals=None, margins=None, noise=None):
+    """Logits [T, vocab]; residuals: a list that receives the stream after every layer; margins: one that receives every
+    router's route_margin; noise: called on every norm's output (to ask how far rounding of a given width reaches)."""
     eps = cfg["norm"]["eps"]
     noise = noise or (lambda a: a)
     x = np.asarray(W["embed"], F64)[np.asarray(tokens)]
@@ -201,7 +219,7 @@ def forward(cfg, W, tokens, residuals=None, noise=None):
         else:
             y = lightning(m, eps, W, h, pre + "mix.")
         if layer.get("mlp") is not None:
-            y = y + feed_forward(layer["mlp"], W, h, pre + "mlp.")
+            y = y + feed_forward(layer["mlp"], W, h, pre + "mlp.", margins)
         x = x + y
         if residuals is not None:
             residuals.append(x.copy())
