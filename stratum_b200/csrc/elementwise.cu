@@ -385,12 +385,58 @@ __global__ void rmsnorm_heads_kernel(T* x, int n_rows, int stride, int first_col
   for (int d = lane; d < head_dim; d += 32) p[d] = from_float<T>(ld_fresh(p + d) * scale * gain[d]);
 }
 
+// The same for wide bfloat16 stretches in multiples of eight values, 16-byte aligned: a block per (row, head), the stretch in
+// registers between its sum and its result.
+#define RH_THREADS 128
+#define RH_PIECES 4
+__global__ void __launch_bounds__(RH_THREADS) rmsnorm_heads_wide_kernel(bf16* x, int stride, int first_col, int n_heads, int head_dim,
+                                                                         const float* __restrict__ gain, float eps) {
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();
+  bf16* p = x + (size_t)(blockIdx.x / n_heads) * stride + first_col + (size_t)(blockIdx.x % n_heads) * head_dim;
+  uint4 v[RH_PIECES];
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < RH_PIECES; u++) {
+    const int d = 8 * (threadIdx.x + RH_THREADS * u);
+    v[u] = d < head_dim ? ld_fresh(reinterpret_cast<const uint4*>(p + d)) : make_uint4(0, 0, 0, 0);
+  }
+#pragma unroll
+  for (int u = 0; u < RH_PIECES; u++) {
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v[u]);
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      const float a = __low2float(h[i]), b = __high2float(h[i]);
+      ss = fmaf(b, b, fmaf(a, a, ss));
+    }
+  }
+  ss = block_sum(ss, scratch);
+  const float scale = 1.0f / sqrtf(ss / (float)head_dim + eps);
+#pragma unroll
+  for (int u = 0; u < RH_PIECES; u++) {
+    const int d = 8 * (threadIdx.x + RH_THREADS * u);
+    if (d >= head_dim) continue;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&v[u]);
+    const float4 g0 = *reinterpret_cast<const float4*>(gain + d), g1 = *reinterpret_cast<const float4*>(gain + d + 4);
+    const float g[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+      h[i] = __floats2bfloat162_rn(__low2float(h[i]) * scale * g[2 * i], __high2float(h[i]) * scale * g[2 * i + 1]);
+    *reinterpret_cast<uint4*>(p + d) = v[u];
+  }
+}
+
 STRATUM_EXPORT int stratum_rmsnorm_heads(void* x, int dtype, int n_rows, int stride, int first_col, int n_heads,
                                          int head_dim, const float* gain, float eps, cudaStream_t stream) {
   if (n_rows <= 0 || n_heads <= 0) return 0;
   if (head_dim <= 0 || first_col < 0 || first_col + (long long)n_heads * head_dim > stride) return STRATUM_ERR_SHAPE;
   const int warps = 4;
   const int blocks = (int)(((long long)n_rows * n_heads + warps - 1) / warps);
+  if (dtype == STRATUM_DT_BF16 && head_dim >= 256 && head_dim <= 8 * RH_THREADS * RH_PIECES && head_dim % 8 == 0 &&
+      first_col % 8 == 0 && stride % 8 == 0 && (((uintptr_t)x | (uintptr_t)gain) & 15) == 0)
+    return launch_pdl(rmsnorm_heads_wide_kernel, n_rows * n_heads, RH_THREADS, 0, stream, (bf16*)x, stride, first_col, n_heads,
+                      head_dim, gain, eps);
   if (dtype == STRATUM_DT_F32)
     return launch_pdl(rmsnorm_heads_kernel<float>, blocks, warps * 32, 0, stream, (float*)x, n_rows, stride,
                       first_col, n_heads, head_dim, gain, eps);

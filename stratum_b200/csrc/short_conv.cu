@@ -41,6 +41,7 @@ struct ShortConv {
 };
 
 #define SC_THREADS 128
+#define SC_BATCH 4            // tokens of a run whose loads are in flight together
 
 template <int VEC> struct ScPack { float v[VEC]; };
 
@@ -108,6 +109,10 @@ __global__ void __launch_bounds__(SC_THREADS) short_conv_kernel(const ShortConv 
   for (int j = 0; j < TAPS; j++)
 #pragma unroll
     for (int e = 0; e < VEC; e++) w[j].v[e] = P.conv_w[(size_t)j * channels + c + e];
+  const bool writes = P.write_cache && seq >= 0;
+  const int* bt = writes && part > 0 ? P.block_table + (size_t)seq * P.bt_stride : nullptr;
+  const int pos0 = P.token_pos[row0];
+  int page_of = pos0 / P.page_tokens, page = bt ? bt[page_of] : -1;      // the page looked up last
   pdl_wait();              // the projection, the state and the first values are the work of kernels before this one
   if (n <= 0) return;      // an entry of a list of fixed length that holds no token
   // the input `back` tokens in front of row i of the run
@@ -124,54 +129,65 @@ __global__ void __launch_bounds__(SC_THREADS) short_conv_kernel(const ShortConv 
     for (int j = 0; j < TAPS - 1; j++) hist[j] = input(0, TAPS - 1 - j);
   }
   const float lam = part == 2 && P.v_first_in ? *P.lambda : 0.f;
-  const bool writes = P.write_cache && seq >= 0;
-  const int* bt = writes && part > 0 ? P.block_table + (size_t)seq * P.bt_stride : nullptr;
-  const int pos0 = P.token_pos[row0];
-#pragma unroll 4
-  for (int i = 0; i < n; i++) {
-    ScPack<VEC> y;
-    if (TAPS > 0) {
-      const ScPack<VEC> u = sc_load<VEC>(in + (size_t)i * P.ld);
+  for (int i0 = 0; i0 < n; i0 += SC_BATCH) {
+    // a batch's loads go out together
+    ScPack<VEC> u[SC_BATCH], first[SC_BATCH];
+    if (TAPS > 0 || taps == 0) {
 #pragma unroll
-      for (int e = 0; e < VEC; e++) {
-        float acc = 0.f;
-#pragma unroll
-        for (int j = 0; j < TAPS - 1; j++) acc = fmaf(w[j].v[e], hist[j].v[e], acc);      // oldest input first
-        y.v[e] = fmaf(w[TAPS > 0 ? TAPS - 1 : 0].v[e], u.v[e], acc);
-      }
-#pragma unroll
-      for (int j = 0; j + 1 < TAPS - 1; j++) hist[j] = hist[j + 1];
-      if (TAPS > 1) hist[TAPS > 1 ? TAPS - 2 : 0] = u;
-    } else if (taps == 0) {
-      y = sc_load<VEC>(in + (size_t)i * P.ld);
-    } else {
-#pragma unroll
-      for (int e = 0; e < VEC; e++) y.v[e] = 0.f;
-      for (int j = 0; j < taps; j++) {
-        const ScPack<VEC> u = input(i, taps - 1 - j);
-#pragma unroll
-        for (int e = 0; e < VEC; e++) y.v[e] = fmaf(P.conv_w[(size_t)j * channels + c + e], u.v[e], y.v[e]);
-      }
+      for (int b = 0; b < SC_BATCH; b++)
+        if (i0 + b < n) u[b] = sc_load<VEC>(in + (size_t)(i0 + b) * P.ld);
     }
-    const size_t row = (size_t)(row0 + i);
-    if (part == 0) {
-      sc_store<VEC>((T*)P.q_out + row * P.ldq + col, y);
-      continue;
-    }
-    if (part == 2) {
-      if (P.v_first_in) {
-        const ScPack<VEC> first = sc_load<VEC>((const T*)P.v_first_in + row * P.ld_first + col);
+    if (part == 2 && P.v_first_in) {
 #pragma unroll
-        for (int e = 0; e < VEC; e++) y.v[e] = (1.0f - lam) * y.v[e] + lam * first.v[e];
-      }
-      if (P.v_first_out) sc_store<VEC>((T*)P.v_first_out + row * P.ld_first + col, y);
+      for (int b = 0; b < SC_BATCH; b++)
+        if (i0 + b < n) first[b] = sc_load<VEC>((const T*)P.v_first_in + (size_t)(row0 + i0 + b) * P.ld_first + col);
     }
-    if (!writes) continue;
-    const int pos = pos0 + i;
-    const int page = bt[pos / P.page_tokens];
-    if (page < 0) continue;
-    T* cache = (T*)(part == 1 ? P.k_cache : P.v_cache);
-    sc_store<VEC>(cache + (((size_t)page * P.n_kv + head) * P.page_tokens + pos % P.page_tokens) * size + d, y);
+#pragma unroll
+    for (int b = 0; b < SC_BATCH; b++) {
+      const int i = i0 + b;
+      if (i >= n) break;
+      ScPack<VEC> y;
+      if (TAPS > 0) {
+#pragma unroll
+        for (int e = 0; e < VEC; e++) {
+          float acc = 0.f;
+#pragma unroll
+          for (int j = 0; j < TAPS - 1; j++) acc = fmaf(w[j].v[e], hist[j].v[e], acc);      // oldest input first
+          y.v[e] = fmaf(w[TAPS > 0 ? TAPS - 1 : 0].v[e], u[b].v[e], acc);
+        }
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS - 1; j++) hist[j] = hist[j + 1];
+        if (TAPS > 1) hist[TAPS > 1 ? TAPS - 2 : 0] = u[b];
+      } else if (taps == 0) {
+        y = u[b];
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; e++) y.v[e] = 0.f;
+        for (int j = 0; j < taps; j++) {
+          const ScPack<VEC> x = input(i, taps - 1 - j);
+#pragma unroll
+          for (int e = 0; e < VEC; e++) y.v[e] = fmaf(P.conv_w[(size_t)j * channels + c + e], x.v[e], y.v[e]);
+        }
+      }
+      const size_t row = (size_t)(row0 + i);
+      if (part == 0) {
+        sc_store<VEC>((T*)P.q_out + row * P.ldq + col, y);
+        continue;
+      }
+      if (part == 2) {
+        if (P.v_first_in) {
+#pragma unroll
+          for (int e = 0; e < VEC; e++) y.v[e] = (1.0f - lam) * y.v[e] + lam * first[b].v[e];
+        }
+        if (P.v_first_out) sc_store<VEC>((T*)P.v_first_out + row * P.ld_first + col, y);
+      }
+      if (!writes) continue;
+      const int pos = pos0 + i, nth = pos / P.page_tokens;
+      if (nth != page_of) { page_of = nth; page = bt[nth]; }
+      if (page < 0) continue;
+      T* cache = (T*)(part == 1 ? P.k_cache : P.v_cache);
+      sc_store<VEC>(cache + (((size_t)page * P.n_kv + head) * P.page_tokens + (pos - nth * P.page_tokens)) * size + d, y);
+    }
   }
   // the sequence's first run moves its state on: row r becomes what stands `len` places further in (state, then the
   // step's tokens); rows are read ahead of where they are written

@@ -57,7 +57,8 @@ def test_rmsnorm_many_rows(dtype, hidden):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("n_heads,head_dim,first", [(5, 48, 0), (2, 128, 640), (7, 20, 8)])
+@pytest.mark.parametrize("n_heads,head_dim,first", [(5, 48, 0), (2, 128, 640), (7, 20, 8), (3, 256, 8), (1, 1536, 64), (2, 600, 16), (1, 4096, 8),
+                                                    (1, 1530, 64), (2, 264, 4)])
 def test_rmsnorm_heads_in_place(dtype, n_heads, head_dim, first):
     """The per-head norm of queries or keys: only the named stretch of each row changes."""
     from stratum_b200 import kernels as K
